@@ -808,3 +808,134 @@ class ZavizenConfig:
         if self.eos_token_id:
             out["eos_token_id"] = list(self.eos_token_id)
         return out
+
+
+@dataclass(frozen=True)
+class LigiraxLayer:
+    """One layer of a Ligirax model as config.json gives it: ``type`` names the mixer, ``mixer`` holds its sizes and
+    constants, ``mlp`` the feed-forward's (None: the layer has none)."""
+
+    type: str
+    mixer: dict
+    mlp: dict | None
+
+    MIXERS = ("latent_attention",)
+
+
+@dataclass(frozen=True)
+class LigiraxConfig:
+    """config.json of the ``Ligirax`` decoder: ``vocab``, ``width``, ``norm.eps``, ``residual_mult`` (what every
+    sublayer's normed result is multiplied by before it joins the stream), ``logit_scale`` and a list of layers.  A
+    layer names its mixer (``latent_attention``: ``heads``, ``dim``, ``rot_dim``, ``vdim``, ``kv_rank``, ``scale``,
+    ``rot`` with ``base``, ``dims`` and an optional ``scaling`` (``factor``, ``original``, ``fast``, ``slow``), an
+    optional window ``mask.size``, and ``kv_from``, an earlier layer whose latents it reads instead of its own) and its
+    feed-forward (``moe`` with ``expert`` (``ff``, ``limit``) and ``router`` (``experts``, ``top``, ``identity``); or
+    null).  Every size and constant is read from here."""
+
+    vocab: int
+    width: int
+    norm_eps: float
+    residual_mult: float
+    logit_scale: float
+    layers: tuple[LigiraxLayer, ...]
+    max_position_embeddings: int = 1 << 20
+    eos_token_id: tuple[int, ...] = ()
+    architectures: tuple[str, ...] = ("Ligirax",)
+
+    ARCHITECTURE = "Ligirax"
+
+    @property
+    def vocab_size(self) -> int:
+        return self.vocab
+
+    @staticmethod
+    def _check_mixer(m: dict, where: str, index: int, earlier: list[LigiraxLayer]) -> None:
+        for key in ("heads", "dim", "rot_dim", "vdim", "kv_rank"):
+            _sized(m, key, where)
+        _number(m, "scale", where)
+        rot, where_r = _section(m, "rot", where), where + "rot: "
+        dims = _sized(rot, "dims", where_r)
+        if _number(rot, "base", where_r) <= 1:
+            raise ConfigError(f"config.json: {where_r}'base' must be above 1")
+        if dims % 2 or dims > m["rot_dim"]:
+            raise ConfigError(f"config.json: {where_r}'dims' must be even and at most 'rot_dim' ({m['rot_dim']}), "
+                              f"got {dims}")
+        if rot.get("scaling") is not None:
+            s = _section(rot, "scaling", where_r)
+            for key in ("factor", "original", "fast", "slow"):
+                if _number(s, key, where_r + "scaling: ") <= 0:
+                    raise ConfigError(f"config.json: {where_r}scaling: '{key}' must be positive")
+        if m.get("mask") is not None:
+            _sized(_section(m, "mask", where), "size", where + "mask: ")
+        source = m.get("kv_from")
+        if source is not None:
+            ok = isinstance(source, int) and not isinstance(source, bool) and 0 <= source < index
+            if not ok or earlier[source].mixer.get("kv_from") is not None:
+                raise ConfigError(f"config.json: {where}'kv_from' must name an earlier layer that has latents of its "
+                                  f"own, got {source!r}")
+            if any(earlier[source].mixer[key] != m[key] for key in ("kv_rank", "rot_dim", "rot")):
+                raise ConfigError(f"config.json: {where}'kv_from': layer {source} keeps latents of another rank or "
+                                  f"turned in another way")
+
+    @staticmethod
+    def _check_mlp(mlp: dict, where: str) -> None:
+        if mlp.get("kind", "moe") != "moe":
+            raise ConfigError(f"config.json: {where}'kind' must be 'moe', got {mlp.get('kind')!r}")
+        expert = _section(mlp, "expert", where)
+        _sized(expert, "ff", where + "expert: ")
+        if _number(expert, "limit", where + "expert: ") <= 0:
+            raise ConfigError(f"config.json: {where}expert: 'limit' must be positive")
+        router, where_r = _section(mlp, "router", where), where + "router: "
+        experts, top = _sized(router, "experts", where_r), _sized(router, "top", where_r)
+        identity = router.get("identity") or 0
+        if isinstance(identity, bool) or not isinstance(identity, int) or identity < 0:
+            raise ConfigError(f"config.json: {where_r}'identity' must be a non-negative integer, got {identity!r}")
+        if top > experts + identity:
+            raise ConfigError(f"config.json: {where_r}'top' ({top}) is more than the {experts} experts and {identity} "
+                              f"identity choices there are")
+
+    @classmethod
+    def from_dict(cls, d: dict[str, Any]) -> "LigiraxConfig":
+        layers_raw = d.get("layers")
+        if not isinstance(layers_raw, (list, tuple)) or not layers_raw:
+            raise ConfigError("config.json: key 'layers' must be a non-empty list")
+        layers: list[LigiraxLayer] = []
+        for i, entry in enumerate(layers_raw):
+            where = f"layers[{i}]: "
+            if not isinstance(entry, dict) or entry.get("type") not in LigiraxLayer.MIXERS:
+                raise ConfigError(f"config.json: {where}'type' must be one of {list(LigiraxLayer.MIXERS)}, "
+                                  f"got {entry.get('type') if isinstance(entry, dict) else entry!r}")
+            mixer = _section(entry, "mixer", where)
+            cls._check_mixer(mixer, where + "mixer: ", i, layers)
+            mlp = entry.get("mlp")
+            if mlp is not None:
+                if not isinstance(mlp, dict):
+                    raise ConfigError(f"config.json: {where}'mlp' must be an object or null")
+                cls._check_mlp(mlp, where + "mlp: ")
+            layers.append(LigiraxLayer(entry["type"], copy.deepcopy(mixer), None if mlp is None else copy.deepcopy(mlp)))
+        eos = d.get("eos_token_id")
+        eos = () if eos is None else ((eos,) if isinstance(eos, int) else tuple(eos))
+        cfg = cls(
+            vocab=_sized(d, "vocab", ""),
+            width=_sized(d, "width", ""),
+            norm_eps=_number(_section(d, "norm", ""), "eps", "norm: "),
+            residual_mult=_number(d, "residual_mult", ""),
+            logit_scale=_number(d, "logit_scale", ""),
+            layers=tuple(layers),
+            max_position_embeddings=_optional(d, "max_position_embeddings", int, 1 << 20),
+            eos_token_id=eos,
+        )
+        if cfg.norm_eps <= 0:
+            raise ConfigError("config.json: norm: 'eps' must be positive")
+        return cfg
+
+    def to_dict(self) -> dict[str, Any]:
+        out = {"architecture": self.ARCHITECTURE, "vocab": self.vocab, "width": self.width,
+               "norm": {"eps": self.norm_eps}, "residual_mult": self.residual_mult, "logit_scale": self.logit_scale,
+               "layers": [{"type": l.type, "mixer": copy.deepcopy(l.mixer),
+                           "mlp": None if l.mlp is None else copy.deepcopy(l.mlp)} for l in self.layers]}
+        if self.max_position_embeddings != 1 << 20:
+            out["max_position_embeddings"] = self.max_position_embeddings
+        if self.eos_token_id:
+            out["eos_token_id"] = list(self.eos_token_id)
+        return out

@@ -885,37 +885,61 @@ void head_prep(const Tensor& x, const OptTensor& slots, Tensor& q_out, const Opt
   check_launch(akv::launch_head_prep(p, stream_of(x)), "head_prep");
 }
 
-void latent_prep(const Tensor& x, const Tensor& positions, const OptTensor& slots, const Tensor& q_weight,
-                 const Tensor& kv_weight, const Tensor& inv_freq, Tensor& q_latent, const OptTensor& cache,
+void latent_prep(const Tensor& x, const Tensor& positions, const OptTensor& slots, const OptTensor& q_weight,
+                 const OptTensor& kv_weight, const Tensor& inv_freq, const OptTensor& q_latent, const OptTensor& cache,
                  int64_t q_rank, int64_t kv_rank, int64_t rot_dim, int64_t rotary_dims, double eps,
-                 const OptTensor& status) {
+                 const OptTensor& status, double factor, const OptTensor& q_rows, int64_t heads, int64_t head_dim,
+                 bool has_kv, const OptTensor& gate) {
   check_cuda(x, "x");
-  check_cuda(q_latent, "q_latent");
-  check_same(x, q_latent, "x", "q_latent");
-  AKV_CHECK(q_rank > 0 && kv_rank > 0 && rot_dim >= 0 && rotary_dims >= 0 && rotary_dims <= rot_dim &&
-                rotary_dims % 2 == 0,
-            "latent_prep: ranks must be positive and rotary_dims an even number up to rot_dim");
-  AKV_CHECK(x.dim() == 2 && x.size(1) == q_rank + kv_rank + rot_dim,
-            "x must be [tokens, q_rank + kv_rank + rot_dim]");
+  AKV_CHECK(q_rank >= 0 && kv_rank > 0 && rot_dim >= 0 && rot_dim <= 1024 && rotary_dims >= 0 &&
+                rotary_dims <= rot_dim && rotary_dims % 2 == 0,
+            "latent_prep: ranks must be positive and rotary_dims an even number up to rot_dim (at most 1024)");
+  AKV_CHECK((q_rank > 0) == q_latent.has_value() && (q_rank > 0) == q_weight.has_value() && !(q_rank > 0 && q_rows.has_value()),
+            "latent_prep: a query latent comes with its weight and output, query heads take its place");
+  AKV_CHECK(q_rank > 0 || q_rows.has_value(), "latent_prep: x begins with a query latent or with query heads");
+  AKV_CHECK(!(q_rows.has_value() || gate.has_value()) || (heads > 0 && head_dim >= 0), "latent_prep: heads must be positive");
+  const int64_t q_cols = q_rank > 0 ? q_rank : heads * (head_dim + rot_dim);
+  const int64_t kv_cols = has_kv ? kv_rank + rot_dim : 0;
+  AKV_CHECK(x.dim() == 2 && x.size(1) >= q_cols + kv_cols + (gate.has_value() ? heads : 0),
+            "x must be [tokens, queries | key/value latent, rotated part | gates]");
   const int64_t n = x.size(0);
   check_i32(positions, "positions", n);
-  check_f32(q_weight, "q_weight", q_rank);
-  check_f32(kv_weight, "kv_weight", kv_rank);
   check_f32(inv_freq, "inv_freq", rotary_dims / 2);
-  AKV_CHECK(q_latent.numel() == n * q_rank, "q_latent must be [tokens, q_rank]");
   akv::LatentPrepParams p{};
   p.x = x.data_ptr();
+  p.x_width = x.size(1);
   p.positions = positions.data_ptr<int>();
   if (slots.has_value()) {
     check_i32(*slots, "slots", n);
     p.slots = slots->data_ptr<int>();
   }
-  p.q_weight = q_weight.data_ptr<float>();
-  p.kv_weight = kv_weight.data_ptr<float>();
+  if (q_rank > 0) {
+    check_cuda(*q_latent, "q_latent");
+    check_same(x, *q_latent, "x", "q_latent");
+    check_f32(*q_weight, "q_weight", q_rank);
+    AKV_CHECK(q_latent->numel() == n * q_rank, "q_latent must be [tokens, q_rank]");
+    p.q_weight = q_weight->data_ptr<float>();
+    p.q_latent = q_latent->data_ptr();
+  } else {
+    check_cuda(*q_rows, "q_rows");
+    check_same(x, *q_rows, "x", "q_rows");
+    AKV_CHECK(q_rows->numel() == n * heads * (kv_rank + rot_dim), "q_rows must be [tokens, heads * (kv_rank + rot_dim)]");
+    p.q_rows = q_rows->data_ptr();
+  }
+  p.heads = (int)heads;
+  p.head_dim = (int)head_dim;
+  p.kv_off = (int)q_cols;
+  p.gate_off = (int)(q_cols + kv_cols);
+  if (gate.has_value()) {
+    check_f32(*gate, "gate", n * heads);
+    p.gate = gate->data_ptr<float>();
+  }
   p.inv_freq = inv_freq.data_ptr<float>();
-  p.q_latent = q_latent.data_ptr();
+  p.factor = (float)factor;
   if (cache.has_value()) {
-    AKV_CHECK(slots.has_value(), "cache needs slots");
+    AKV_CHECK(slots.has_value() && has_kv && kv_weight.has_value(), "cache needs slots, key/value columns and kv_weight");
+    check_f32(*kv_weight, "kv_weight", kv_rank);
+    p.kv_weight = kv_weight->data_ptr<float>();
     check_pages(*cache, "cache", 1, kv_rank + rot_dim, x);
     p.cache = cache->data_ptr();
     p.page_size = (int)cache->size(2);
@@ -935,7 +959,7 @@ void latent_prep(const Tensor& x, const Tensor& positions, const OptTensor& slot
 }
 
 void rotate_pairs(const Tensor& in, Tensor& out, const Tensor& positions, const Tensor& inv_freq, int64_t heads,
-                  int64_t cols, int64_t rotary_dims, int64_t in_offset, int64_t out_offset) {
+                  int64_t cols, int64_t rotary_dims, int64_t in_offset, int64_t out_offset, double factor) {
   check_cuda(in, "in");
   check_cuda(out, "out");
   check_same(in, out, "in", "out");
@@ -951,8 +975,8 @@ void rotate_pairs(const Tensor& in, Tensor& out, const Tensor& positions, const 
   c10::cuda::CUDAGuard guard(in.device());
   check_launch(akv::launch_rotate_pairs(in.data_ptr(), out.data_ptr(), positions.data_ptr<int>(),
                                         inv_freq.data_ptr<float>(), n, (int)heads, (int)cols, (int)rotary_dims,
-                                        in_width, (int)in_offset, out_width, (int)out_offset, dtype_code(in, "in"),
-                                        stream_of(in)),
+                                        in_width, (int)in_offset, out_width, (int)out_offset, (float)factor,
+                                        dtype_code(in, "in"), stream_of(in)),
                "rotate_pairs");
 }
 
@@ -1057,6 +1081,71 @@ void branch_layernorm_parts(Tensor& hidden, const Tensor& parts, const OptTensor
                                                   shared_code, weight.data_ptr<float>(), copy_ptr, copy_code, n, h,
                                                   (float)eps, stream_of(hidden)),
                "branch_layernorm_parts");
+}
+
+// hidden += norm(branch) * weight, then the stream's own norm into out (see launchers.h).  The branch is `branch`, or
+// `parts` with `top` rows per token (and `chosen` / `pair_weights` / `x` where choices from first_identity on are the
+// identity).
+void branch_rmsnorm(Tensor& hidden, const OptTensor& branch, const OptTensor& parts, const OptTensor& shared, int64_t top,
+                    const OptTensor& chosen, const OptTensor& pair_weights, const OptTensor& x, int64_t first_identity,
+                    const Tensor& weight, double eps, const OptTensor& next_weight, double next_eps,
+                    const OptTensor& out, const OptTensor& rows, const OptTensor& status) {
+  check_cuda(hidden, "hidden");
+  AKV_CHECK(hidden.scalar_type() == at::kFloat && hidden.dim() == 2, "hidden must be float32 [tokens, hidden]");
+  const int64_t n = hidden.size(0), h = hidden.size(1);
+  AKV_CHECK(h * 4 <= 200 * 1024, "branch_rmsnorm: hidden size ", h, " exceeds the kernel's limit of 51200");
+  AKV_CHECK(branch.has_value() != parts.has_value(), "branch_rmsnorm: either branch or parts");
+  auto row_tensor = [&](const OptTensor& t, const char* name, int& code) -> const void* {
+    check_cuda(*t, name);
+    AKV_CHECK(t->numel() == n * h && t->device() == hidden.device(), name, " must be [tokens, hidden]");
+    code = dtype_code(*t, name);
+    return t->data_ptr();
+  };
+  check_f32(weight, "weight", h);
+  akv::BranchNormParams p{};
+  p.hidden = hidden.data_ptr<float>();
+  p.weight = weight.data_ptr<float>();
+  p.eps = (float)eps;
+  if (branch.has_value()) {
+    p.branch = row_tensor(branch, "branch", p.branch_dtype);
+  } else {
+    AKV_CHECK(top >= 1 && top <= akv::kBranchNormMaxTop, "branch_rmsnorm: top must be between 1 and 32, got ", top);
+    check_f32(*parts, "parts", n * top * h);
+    p.parts = parts->data_ptr<float>();
+    p.top = (int)top;
+    if (shared.has_value()) p.shared = row_tensor(shared, "shared", p.shared_dtype);
+    if (chosen.has_value()) {
+      AKV_CHECK(pair_weights.has_value() && x.has_value(), "branch_rmsnorm: chosen comes with pair_weights and x");
+      check_i32(*chosen, "chosen", n * top);
+      check_f32(*pair_weights, "pair_weights", n * top);
+      p.chosen = chosen->data_ptr<int>();
+      p.pair_weights = pair_weights->data_ptr<float>();
+      p.x = row_tensor(x, "x", p.x_dtype);
+      p.first_identity = (int)first_identity;
+    }
+  }
+  AKV_CHECK(next_weight.has_value() == out.has_value(), "branch_rmsnorm: next_weight and out go together");
+  int64_t out_rows = n;
+  if (rows.has_value()) {
+    check_i32(*rows, "rows");
+    AKV_CHECK(out.has_value(), "branch_rmsnorm: rows need an output");
+    p.rows = rows->data_ptr<int>();
+    p.num_rows = out_rows = rows->numel();
+  }
+  if (out.has_value()) {
+    check_f32(*next_weight, "next_weight", h);
+    check_cuda(*out, "out");
+    AKV_CHECK(out->numel() == out_rows * h && out->device() == hidden.device(), "out must be [rows, hidden]");
+    p.next_weight = next_weight->data_ptr<float>();
+    p.out = out->data_ptr();
+    p.out_dtype = dtype_code(*out, "out");
+  }
+  p.next_eps = (float)next_eps;
+  p.num_tokens = n;
+  p.width = (int)h;
+  p.status = status_ptr(status);
+  c10::cuda::CUDAGuard guard(hidden.device());
+  check_launch(akv::launch_branch_rmsnorm(p, stream_of(hidden)), "branch_rmsnorm");
 }
 
 void stream_copy(const Tensor& hidden, Tensor& out) {
@@ -1654,7 +1743,8 @@ void conv_tail(const Tensor& x, Tensor& state, int64_t tail_off, const Tensor& c
 }
 
 void moe_route(const Tensor& logits, const OptTensor& correction, Tensor& chosen, Tensor& weights, int64_t groups,
-               int64_t keep_groups, int64_t group_top, double scale, double weight_eps, int64_t score_kind) {
+               int64_t keep_groups, int64_t group_top, double scale, double weight_eps, int64_t score_kind,
+               bool normalize) {
   check_cuda(logits, "logits");
   AKV_CHECK(logits.scalar_type() == at::kFloat && logits.dim() == 2, "logits must be float32 [tokens, experts]");
   const int64_t n = logits.size(0), experts = logits.size(1);
@@ -1685,6 +1775,7 @@ void moe_route(const Tensor& logits, const OptTensor& correction, Tensor& chosen
   p.weight_eps = (float)weight_eps;
   AKV_CHECK(score_kind == 0 || score_kind == 1, "moe_route: score_kind 0 (sigmoid) or 1 (softmax)");
   p.score_kind = (int)score_kind;
+  p.normalize = normalize ? 1 : 0;
   c10::cuda::CUDAGuard guard(logits.device());
   check_launch(akv::launch_moe_route(p, stream_of(logits)), "moe_route");
 }
@@ -1780,7 +1871,8 @@ void moe_down(const Tensor& act, const Tensor& w, const Tensor& order, const Ten
   check_launch(akv::launch_moe_gemm(p, false, stream_of(act)), "moe_down");
 }
 
-void moe_combine(const Tensor& parts, const OptTensor& shared, Tensor& out, int64_t top) {
+void moe_combine(const Tensor& parts, const OptTensor& shared, Tensor& out, int64_t top, const OptTensor& chosen,
+                 const OptTensor& pair_weights, const OptTensor& x, int64_t first_identity) {
   check_cuda(parts, "parts");
   AKV_CHECK(parts.scalar_type() == at::kFloat && parts.dim() == 2 && top >= 1 && parts.size(0) % top == 0,
             "moe_combine: parts must be float32 [tokens * top, hidden]");
@@ -1795,8 +1887,24 @@ void moe_combine(const Tensor& parts, const OptTensor& shared, Tensor& out, int6
     shared_code = dtype_code(*shared, "shared");
   }
   c10::cuda::CUDAGuard guard(parts.device());
+  const int* chosen_ptr = nullptr;
+  const float* weights_ptr = nullptr;
+  const void* x_ptr = nullptr;
+  int x_code = 0;
+  if (chosen.has_value()) {
+    AKV_CHECK(pair_weights.has_value() && x.has_value(), "moe_combine: chosen comes with pair_weights and x");
+    check_i32(*chosen, "chosen", n * top);
+    check_f32(*pair_weights, "pair_weights", n * top);
+    check_cuda(*x, "x");
+    AKV_CHECK(x->numel() == n * h && x->device() == parts.device(), "x must be [tokens, hidden]");
+    chosen_ptr = chosen->data_ptr<int>();
+    weights_ptr = pair_weights->data_ptr<float>();
+    x_ptr = x->data_ptr();
+    x_code = dtype_code(*x, "x");
+  }
   check_launch(akv::launch_moe_combine(parts.data_ptr<float>(), shared_ptr, shared_code, out.data_ptr<float>(), n, h,
-                                       (int)top, stream_of(parts)),
+                                       (int)top, chosen_ptr, weights_ptr, x_ptr, x_code, (int)first_identity,
+                                       stream_of(parts)),
                "moe_combine");
 }
 
@@ -1881,9 +1989,16 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("k_weight") = py::none(), py::arg("has_kv") = true);
   m.def("latent_prep", &latent_prep, py::arg("x"), py::arg("positions"), py::arg("slots"), py::arg("q_weight"),
         py::arg("kv_weight"), py::arg("inv_freq"), py::arg("q_latent"), py::arg("cache"), py::arg("q_rank"),
-        py::arg("kv_rank"), py::arg("rot_dim"), py::arg("rotary_dims"), py::arg("eps"), py::arg("status") = py::none());
+        py::arg("kv_rank"), py::arg("rot_dim"), py::arg("rotary_dims"), py::arg("eps"), py::arg("status") = py::none(),
+        py::arg("factor") = 1.0, py::arg("q_rows") = py::none(), py::arg("heads") = 0, py::arg("head_dim") = 0,
+        py::arg("has_kv") = true, py::arg("gate") = py::none());
   m.def("rotate_pairs", &rotate_pairs, py::arg("in"), py::arg("out"), py::arg("positions"), py::arg("inv_freq"),
-        py::arg("heads"), py::arg("cols"), py::arg("rotary_dims"), py::arg("in_offset"), py::arg("out_offset"));
+        py::arg("heads"), py::arg("cols"), py::arg("rotary_dims"), py::arg("in_offset"), py::arg("out_offset"),
+        py::arg("factor") = 1.0);
+  m.def("branch_rmsnorm", &branch_rmsnorm, py::arg("hidden"), py::arg("branch"), py::arg("parts"), py::arg("shared"),
+        py::arg("top"), py::arg("chosen"), py::arg("pair_weights"), py::arg("x"), py::arg("first_identity"),
+        py::arg("weight"), py::arg("eps"), py::arg("next_weight"), py::arg("next_eps"), py::arg("out"),
+        py::arg("rows") = py::none(), py::arg("status") = py::none());
   m.def("activation", &activation, py::arg("in"), py::arg("out"), py::arg("kind"));
   m.def("add_layernorm", &add_layernorm, py::arg("hidden"), py::arg("delta"), py::arg("weight"), py::arg("out"),
         py::arg("rows"), py::arg("eps"), py::arg("status") = py::none());
@@ -1946,14 +2061,16 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("scaled_sum", &scaled_sum, py::arg("a"), py::arg("b"), py::arg("out"), py::arg("sa"), py::arg("sb"));
   m.def("moe_route", &moe_route, py::arg("logits"), py::arg("correction"), py::arg("chosen"), py::arg("weights"),
         py::arg("groups"), py::arg("keep_groups"), py::arg("group_top"), py::arg("scale"), py::arg("weight_eps"),
-        py::arg("score_kind") = 0);
+        py::arg("score_kind") = 0, py::arg("normalize") = true);
   m.def("moe_router", &moe_router, py::arg("x"), py::arg("w"), py::arg("logits"));
   m.def("moe_sort", &moe_sort, py::arg("chosen"), py::arg("order"), py::arg("offsets"));
   m.def("moe_gate_up", &moe_gate_up, py::arg("x"), py::arg("w"), py::arg("order"), py::arg("offsets"), py::arg("act"),
         py::arg("top"), py::arg("limit"), py::arg("slope"), py::arg("form") = 0, py::arg("up_offset") = 1.0);
   m.def("moe_down", &moe_down, py::arg("act"), py::arg("w"), py::arg("order"), py::arg("offsets"), py::arg("weights"),
         py::arg("out"), py::arg("form") = 0);
-  m.def("moe_combine", &moe_combine, py::arg("parts"), py::arg("shared"), py::arg("out"), py::arg("top"));
+  m.def("moe_combine", &moe_combine, py::arg("parts"), py::arg("shared"), py::arg("out"), py::arg("top"),
+        py::arg("chosen") = py::none(), py::arg("pair_weights") = py::none(), py::arg("x") = py::none(),
+        py::arg("first_identity") = 0);
   m.def("paged_attention", &paged_attention, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("out"),
         py::arg("block_table"), py::arg("cu_q"), py::arg("ctx_lens"), py::arg("tile_seq"), py::arg("tile_q0"),
         py::arg("tile_nq"), py::arg("partials"), py::arg("num_tiles"), py::arg("q_tile"), py::arg("num_splits"),

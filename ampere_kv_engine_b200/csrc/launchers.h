@@ -278,33 +278,68 @@ struct HeadPrepParams {
 };
 int launch_head_prep(const HeadPrepParams& p, cudaStream_t stream);
 
-// What stands between one product that holds [query latent | key/value latent | rotated key part] of every token and
-// what comes next: RMS norm with a plain weight on each latent, rotary positions on neighbouring pairs of the first
-// rotary_dims dims of the rotated part; the normed key/value latent and the rotated part go side by side into the
-// token's cache row [kv_rank + rot_dim].
+// What stands between one product that holds [query latent or query heads | key/value latent | rotated key part | gate
+// columns | unused columns] of every token and what comes next: RMS norm with a plain weight on each latent, rotary
+// positions on neighbouring pairs of the first rotary_dims dims of the rotated part (and of every query head's last
+// rot_dim dims), sigmoid of the gates; the normed key/value latent and the rotated part go side by side into the token's
+// cache row [kv_rank + rot_dim], a query head's turned dims behind the first kv_rank columns of its row of q_rows.
 struct LatentPrepParams {
-  const void* x;               // [N, q_rank + kv_rank + rot_dim]
+  const void* x;               // [N, x_width]
   const int32_t* positions;    // [N]
   const int32_t* slots;        // [N] or null
-  const float* q_weight;       // [q_rank]
-  const float* kv_weight;      // [kv_rank]
+  const float* q_weight;       // [q_rank] or null
+  const float* kv_weight;      // [kv_rank] or null
   const float* inv_freq;       // [rotary_dims / 2]
-  void* q_latent;              // [N, q_rank]
+  void* q_latent;              // [N, q_rank] or null
   void* cache;                 // [num_pages, 1, page_size, row_stride] or null
-  int64_t num_tokens;
+  void* q_rows;                // [N, heads, kv_rank + rot_dim] or null: x then begins with heads * (head_dim + rot_dim)
+                               // query columns in place of a query latent
+  float* gate;                 // [N, heads] or null
+  int64_t num_tokens, x_width;
   int q_rank, kv_rank, rot_dim, rotary_dims, page_size;
+  int heads, head_dim;         // read with q_rows (and heads with gate)
+  int kv_off, gate_off;        // first column of the key/value latent and of the gates
   int64_t num_pages, row_stride;
-  float eps;
+  float eps, factor;           // factor: on cos and sin
   int dtype;
   int* status;
 };
 int launch_latent_prep(const LatentPrepParams& p, cudaStream_t stream);
 
 // out[t, h, out_offset + c] = rotated in[t, h, in_offset + c] for c < cols: dims 2i and 2i + 1 turn by
-// positions[t] * inv_freq[i] while 2i + 1 < rotary_dims, the rest passes unchanged.
+// positions[t] * inv_freq[i] while 2i + 1 < rotary_dims (cos and sin times factor), the rest passes unchanged.
 int launch_rotate_pairs(const void* in, void* out, const int32_t* positions, const float* inv_freq,
                         int64_t num_tokens, int heads, int cols, int rotary_dims, int64_t in_width, int in_offset,
-                        int64_t out_width, int out_offset, int dtype, cudaStream_t stream);
+                        int64_t out_width, int out_offset, float factor, int dtype, cudaStream_t stream);
+
+// A branch's result normed and added to the float32 stream, and the stream's own norm for the next branch, in one pass
+// (sandwich_norm.cu): hidden += b / sqrt(mean(b^2) + eps) * weight, then out = hidden / sqrt(mean(hidden^2) + next_eps)
+// * next_weight.  The branch b is `branch`, or the sum of a token's `top` float32 rows of `parts` in order (plus
+// `shared`), of which those whose choice is `first_identity` or above count as pair weight times the token's row of x.
+struct BranchNormParams {
+  float* hidden;               // [N, width]
+  const void* branch;          // [N, width] or null
+  int branch_dtype;
+  const float* parts;          // [N * top, width] (without branch)
+  int top;
+  const void* shared;          // [N, width] or null
+  int shared_dtype;
+  const int32_t* chosen;       // [N, top] or null: no identity choices
+  const float* pair_weights;   // [N, top]
+  const void* x;               // [N, width]
+  int x_dtype, first_identity;
+  const float* weight;         // [width]
+  const float* next_weight;    // [width] or null: no second norm
+  void* out;                   // [N or num_rows, width] of out_dtype
+  int out_dtype;
+  const int32_t* rows;         // [num_rows] or null: only these rows are made and hidden is left as it is
+  int64_t num_rows, num_tokens;
+  int width;
+  float eps, next_eps;
+  int* status;
+};
+constexpr int kBranchNormMaxTop = 32;
+int launch_branch_rmsnorm(const BranchNormParams& p, cudaStream_t stream);
 
 // The gated delta rule (delta_rule.cu).  x [N, q | k | v | gate | beta | step] with num_kv_heads heads of head_dim
 // for q and k, num_heads heads of v_dim for v and gate, one column per head for beta and step.  state
@@ -347,6 +382,7 @@ struct MoeRouteParams {
   int experts, top, groups, keep_groups, group_top;
   float scale, weight_eps;
   int score_kind;              // 0: sigmoid of each logit; 1: softmax over all experts
+  int normalize;               // 1: the chosen scores are divided by their sum (plus weight_eps)
 };
 int launch_moe_route(const MoeRouteParams& p, cudaStream_t stream);
 // logits[t, e] = x[t, :] . w[e, :] in float, a warp per (token, expert): for steps of a few tokens.
@@ -373,9 +409,11 @@ struct MoeGemmParams {
 // tokens, 64 experts of 1,024 x 4,096: 103 against 111 us; the down product is faster in tiles: 59 against 89 us)
 constexpr int kMoeFewRowPairs = 128;
 int launch_moe_gemm(const MoeGemmParams& p, bool gated, cudaStream_t stream);
-// out[t] = sum over c < top of parts[t * top + c] (+ shared[t]), float32.
+// out[t] = sum over c < top of parts[t * top + c] (+ shared[t]), float32; with `chosen` the choices from
+// first_identity on count as pair_weights[t, c] * x[t].
 int launch_moe_combine(const float* parts, const void* shared, int shared_dtype, float* out, int64_t num_tokens,
-                       int64_t width, int top, cudaStream_t stream);
+                       int64_t width, int top, const int32_t* chosen, const float* pair_weights, const void* x,
+                       int x_dtype, int first_identity, cudaStream_t stream);
 
 enum Activation : int { kActReluSquared = 0, kActGeluTanh = 1, kActSilu = 2 };
 int launch_activation(const void* in, void* out, int64_t total, int kind, int dtype, cudaStream_t stream);

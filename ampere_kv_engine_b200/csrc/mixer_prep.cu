@@ -6,9 +6,10 @@
 //                  q and k heads are scaled to unit RMS (no weight), v is blended with the values an earlier
 //                  layer computed for the same token, k and v go to their cache slots, the gates through a
 //                  sigmoid.
-//   latent_prep:   one product holds [query latent | key/value latent | shared rotated key part].  Both latents
-//                  get an RMS norm with a plain weight; the rotated part gets rotary positions (pairs of
-//                  neighbouring dims); latent and rotated part are written side by side into the token's cache row.
+//   latent_prep:   one product holds [query latent or query heads | key/value latent | shared rotated key part | gates].
+//                  Both latents get an RMS norm with a plain weight; the rotated part and the query heads' rotated dims
+//                  get rotary positions (pairs of neighbouring dims); latent and rotated part are written side by side
+//                  into the token's cache row; the gates go through a sigmoid.
 //   rotate_pairs:  rotary positions on a column range of every head of a [tokens, heads, width] tensor, written to
 //                  a column range of another such tensor.
 //   activation:    relu(x)^2, tanh-form GELU or SiLU, element by element.
@@ -108,25 +109,56 @@ int launch_head_prep(const HeadPrepParams& p, cudaStream_t stream) {
   return (int)launch_chain(head_prep_kernel<float>, dim3((unsigned)blocks), dim3(warps * 32), 0, stream, dim3(1, 1, 1), p);
 }
 
-// One block per (token, segment): 0 = query latent, 1 = key/value latent, 2 = rotated key part.  (A warp per segment
-// walked a latent of several hundred elements in a dozen dependent rounds: 14 us for 8 tokens.)
+namespace {
+
+// dims 2i and 2i + 1 of `src` turned by (cos, sin) and stored at the same place of `dst`; `paired`: both addresses allow
+// one access for the two elements
 template <typename T>
-__global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepParams p) {
+__device__ __forceinline__ void turn_pair(const T* src, T* dst, float cs, float sn, bool paired) {
+  float u, v;
+  if constexpr (sizeof(T) == 2) {
+    if (paired) {
+      const __nv_bfloat162 raw = *reinterpret_cast<const __nv_bfloat162*>(src);
+      u = __low2float(raw);
+      v = __high2float(raw);
+      *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(u * cs - v * sn, v * cs + u * sn);
+      return;
+    }
+  }
+  u = to_float<T>(src[0]);
+  v = to_float<T>(src[1]);
+  dst[0] = from_float<T>(u * cs - v * sn);
+  dst[1] = from_float<T>(v * cs + u * sn);
+}
+
+constexpr int kLatentPrepThreads = 128;
+constexpr int kLatentMaxPairs = 512;         // rotated dims of a head or of the shared key part: up to 1,024
+
+}  // namespace
+
+// One block per (token, unit): the query latent; the key/value latent; the rotated key part and the gates; then the
+// query heads' rotated dims in `q_units` equal groups of heads.  Units a call does not have are not launched: `first`
+// is the number of the first one.  (A warp per latent walked several hundred elements in a dozen dependent rounds: 14 us
+// for 8 tokens.)
+template <typename T>
+__global__ void __launch_bounds__(kLatentPrepThreads) latent_prep_kernel(LatentPrepParams p, int first, int units,
+                                                                         int q_units) {
   __shared__ float scratch[33];
+  __shared__ float2 table[kLatentMaxPairs];
   pdl_launch_dependents();
   pdl_wait();
-  const int64_t token = blockIdx.x / 3;
-  const int segment = (int)(blockIdx.x - token * 3);
-  const int64_t width = (int64_t)p.q_rank + p.kv_rank + p.rot_dim;
-  const T* x = (const T*)p.x + token * width;
+  const int64_t token = blockIdx.x / units;
+  const int unit = first + (int)(blockIdx.x - token * units);
+  const T* x = (const T*)p.x + token * p.x_width;
   const int slot = p.slots != nullptr ? p.slots[token] : -1;
-  T* row = p.cache != nullptr ? cache_row((T*)p.cache, slot, p.page_size, p.num_pages, 1, 0, p.row_stride, p.status)
-                              : nullptr;
-  if (segment < 2) {
-    const int n = segment == 0 ? p.q_rank : p.kv_rank;
-    const T* src = x + (segment == 0 ? 0 : p.q_rank);
-    const float* w = segment == 0 ? p.q_weight : p.kv_weight;
-    T* dst = segment == 0 ? (T*)p.q_latent + token * (int64_t)p.q_rank : row;
+  T* row = nullptr;
+  if (unit >= 1 && unit <= 2 && p.cache != nullptr)
+    row = cache_row((T*)p.cache, slot, p.page_size, p.num_pages, 1, 0, p.row_stride, p.status);
+  if (unit < 2) {
+    const int n = unit == 0 ? p.q_rank : p.kv_rank;
+    const T* src = x + (unit == 0 ? 0 : p.kv_off);
+    const float* w = unit == 0 ? p.q_weight : p.kv_weight;
+    T* dst = unit == 0 ? (T*)p.q_latent + token * (int64_t)p.q_rank : row;
     if (n == 0 || dst == nullptr) return;                  // the same for every thread of the block
     float ss = 0.f;
     for (int d = threadIdx.x; d < n; d += blockDim.x) {
@@ -137,35 +169,76 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepParams p) {
     for (int d = threadIdx.x; d < n; d += blockDim.x) dst[d] = from_float<T>(to_float<T>(src[d]) * inv * w[d]);
     return;
   }
-  if (row == nullptr) return;
-  const T* src = x + p.q_rank + p.kv_rank;
-  T* dst = row + p.kv_rank;
+  const int turning = p.rotary_dims / 2;
   const float position = (float)p.positions[token];
-  const int pairs = p.rot_dim / 2, turning = p.rotary_dims / 2;
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-    float u = to_float<T>(src[2 * i]), v = to_float<T>(src[2 * i + 1]);
-    if (i < turning) {
+  if (unit == 2) {
+    if (p.gate != nullptr)
+      for (int h = threadIdx.x; h < p.heads; h += blockDim.x)
+        p.gate[token * p.heads + h] = 1.f / (1.f + expf(-to_float<T>(x[p.gate_off + h])));
+    if (row == nullptr) return;
+    const T* src = x + p.kv_off + p.kv_rank;
+    T* dst = row + p.kv_rank;
+    for (int i = threadIdx.x; i < turning; i += blockDim.x) {
       float sn, cs;
       sincosf(position * p.inv_freq[i], &sn, &cs);
-      const float a = u * cs - v * sn, b = v * cs + u * sn;
-      u = a;
-      v = b;
+      turn_pair<T>(src + 2 * i, dst + 2 * i, cs * p.factor, sn * p.factor, false);
     }
-    dst[2 * i] = from_float<T>(u);
-    dst[2 * i + 1] = from_float<T>(v);
+    for (int d = p.rotary_dims + threadIdx.x; d < p.rot_dim; d += blockDim.x) dst[d] = src[d];
+    return;
   }
-  if ((p.rot_dim & 1) && threadIdx.x == 0) dst[p.rot_dim - 1] = src[p.rot_dim - 1];
+  // query heads: a table of the token's angles first, then every (head, pair) of the group
+  for (int i = threadIdx.x; i < turning; i += blockDim.x) {
+    float sn, cs;
+    sincosf(position * p.inv_freq[i], &sn, &cs);
+    table[i] = make_float2(cs * p.factor, sn * p.factor);
+  }
+  __syncthreads();
+  const int per = (p.heads + q_units - 1) / q_units;
+  const int h0 = (unit - 3) * per, h1 = min(p.heads, h0 + per);
+  const int in_width = p.head_dim + p.rot_dim, out_width = p.kv_rank + p.rot_dim;
+  T* out = (T*)p.q_rows + token * p.heads * (int64_t)out_width;
+  const bool paired = sizeof(T) == 2 && ((p.x_width | in_width | p.head_dim | out_width | p.kv_rank) & 1) == 0 &&
+                      (reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.q_rows)) % 4 == 0;
+  for (int idx = threadIdx.x; idx < (h1 - h0) * turning; idx += blockDim.x) {
+    const int h = h0 + idx / turning, i = idx % turning;
+    turn_pair<T>(x + (int64_t)h * in_width + p.head_dim + 2 * i, out + (int64_t)h * out_width + p.kv_rank + 2 * i,
+                 table[i].x, table[i].y, paired);
+  }
+  const int still = p.rot_dim - p.rotary_dims;
+  for (int idx = threadIdx.x; idx < (h1 - h0) * still; idx += blockDim.x) {
+    const int h = h0 + idx / still, d = p.rotary_dims + idx % still;
+    out[(int64_t)h * out_width + p.kv_rank + d] = x[(int64_t)h * in_width + p.head_dim + d];
+  }
 }
 
 int launch_latent_prep(const LatentPrepParams& p, cudaStream_t stream) {
   if (p.num_tokens == 0) return 0;
-  if (p.rotary_dims > p.rot_dim || (p.rotary_dims & 1)) return (int)cudaErrorInvalidValue;
-  const int64_t blocks = p.num_tokens * 3;
+  if (p.rotary_dims > p.rot_dim || (p.rotary_dims & 1) || p.rotary_dims / 2 > kLatentMaxPairs ||
+      (p.q_latent != nullptr && p.q_rows != nullptr) || (p.q_rows != nullptr && p.heads <= 0))
+    return (int)cudaErrorInvalidValue;
+  // query heads: one group of heads per token where the tokens fill the GPU, more where they are few
+  int q_units = 0;
+  if (p.q_rows != nullptr && p.rot_dim > 0) {
+    const int64_t most = ((int64_t)p.heads * ((p.rot_dim + 1) / 2) + kLatentPrepThreads - 1) / kLatentPrepThreads;
+    q_units = (int)(256 / p.num_tokens);
+    if (q_units > most) q_units = (int)most;
+    if (q_units > p.heads) q_units = p.heads;
+    if (q_units < 1) q_units = 1;
+  }
+  const bool middle = p.cache != nullptr || p.gate != nullptr;
+  // the units are numbered 0 (query latent), 1, 2 (key/value side and gates), 3 .. (query heads); those launched are
+  // [first, first + units): without a query latent the numbering begins at 1, without a key/value side at 2, ...
+  const int first = p.q_latent != nullptr ? 0 : (p.cache != nullptr ? 1 : (p.gate != nullptr ? 2 : 3));
+  const int last = q_units > 0 ? 3 + q_units : (middle ? 3 : 1);
+  const int units = last - first;
+  if (units <= 0) return 0;
+  const int64_t blocks = p.num_tokens * units;
   if (blocks > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
+  const dim3 grid((unsigned)blocks), block(kLatentPrepThreads);
   if (p.dtype == kBFloat16)
-    return (int)launch_chain(latent_prep_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(128), 0, stream,
-                             dim3(1, 1, 1), p);
-  return (int)launch_chain(latent_prep_kernel<float>, dim3((unsigned)blocks), dim3(128), 0, stream, dim3(1, 1, 1), p);
+    return (int)launch_chain(latent_prep_kernel<__nv_bfloat16>, grid, block, 0, stream, dim3(1, 1, 1), p, first, units,
+                             q_units);
+  return (int)launch_chain(latent_prep_kernel<float>, grid, block, 0, stream, dim3(1, 1, 1), p, first, units, q_units);
 }
 
 // One thread per (token, head, pair of the column range).
@@ -173,7 +246,7 @@ template <typename T>
 __global__ void rotate_pairs_kernel(const T* __restrict__ in, T* __restrict__ out, const int32_t* __restrict__ positions,
                                     const float* __restrict__ inv_freq, int64_t total, int heads, int cols,
                                     int rotary_dims, int64_t in_width, int in_offset, int64_t out_width,
-                                    int out_offset) {
+                                    int out_offset, float factor) {
   pdl_launch_dependents();
   pdl_wait();
   const int pairs = (cols + 1) / 2;
@@ -192,6 +265,8 @@ __global__ void rotate_pairs_kernel(const T* __restrict__ in, T* __restrict__ ou
   if (2 * i + 1 < rotary_dims) {
     float sn, cs;
     sincosf((float)positions[token] * inv_freq[i], &sn, &cs);
+    sn *= factor;
+    cs *= factor;
     const float a = u * cs - v * sn, b = v * cs + u * sn;
     u = a;
     v = b;
@@ -202,7 +277,7 @@ __global__ void rotate_pairs_kernel(const T* __restrict__ in, T* __restrict__ ou
 
 int launch_rotate_pairs(const void* in, void* out, const int32_t* positions, const float* inv_freq,
                         int64_t num_tokens, int heads, int cols, int rotary_dims, int64_t in_width, int in_offset,
-                        int64_t out_width, int out_offset, int dtype, cudaStream_t stream) {
+                        int64_t out_width, int out_offset, float factor, int dtype, cudaStream_t stream) {
   const int64_t total = num_tokens * heads * ((cols + 1) / 2);
   if (total == 0) return 0;
   if (rotary_dims > cols || (rotary_dims & 1) || in_offset + cols > in_width || out_offset + cols > out_width)
@@ -213,10 +288,10 @@ int launch_rotate_pairs(const void* in, void* out, const int32_t* positions, con
   if (dtype == kBFloat16)
     return (int)launch_chain(rotate_pairs_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(threads), 0, stream,
                              dim3(1, 1, 1), (const __nv_bfloat16*)in, (__nv_bfloat16*)out, positions, inv_freq, total,
-                             heads, cols, rotary_dims, in_width, in_offset, out_width, out_offset);
+                             heads, cols, rotary_dims, in_width, in_offset, out_width, out_offset, factor);
   return (int)launch_chain(rotate_pairs_kernel<float>, dim3((unsigned)blocks), dim3(threads), 0, stream, dim3(1, 1, 1),
                            (const float*)in, (float*)out, positions, inv_freq, total, heads, cols, rotary_dims,
-                           in_width, in_offset, out_width, out_offset);
+                           in_width, in_offset, out_width, out_offset, factor);
 }
 
 template <typename T>

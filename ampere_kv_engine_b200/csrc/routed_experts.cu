@@ -4,13 +4,16 @@
 //   moe_route:    per token: s = sigmoid(logits); choice = s + correction; the experts form equal groups of
 //                 neighbours, a group's score is the sum of its group_top largest choice scores, only experts of the
 //                 keep best groups can be chosen; the top largest remaining choice scores are chosen (ties: the lower
-//                 index); weights = chosen s / (their sum + eps) * scale.  One warp per token, all in float.
+//                 index); weights = chosen s / (their sum + eps) * scale, or chosen s * scale.  One warp per token, all
+//                 in float.
 //   moe_sort:     a counting sort of the (token, choice) pairs by expert: where each expert's run begins, and the
 //                 pairs in that order (within an expert in no particular order: every row is computed by itself).
 //   moe_gate_up:  for the sorted rows of every expert, both products with the expert's matrices and the clamped
 //                 activation on the output tile.
 //   moe_down:     the third product, times the pair's weight, written to the pair's own row (float32).
-//   moe_combine:  a token's rows added up in the order of its choices, plus the shared expert's row.
+//   moe_combine:  a token's rows added up in the order of its choices, plus the shared expert's row; choices that
+//                 are the identity (they lie behind the experts: the sort puts their pairs last and no product sees
+//                 them) count as their weight times the token's input.
 //
 // The grouped products tile the sorted rows expert by expert: a block finds its (expert, row tile) by walking the
 // run starts, so the grid depends on the batch layout alone.  Each output element is one dot product accumulated
@@ -140,7 +143,7 @@ __global__ void moe_route_kernel(MoeRouteParams p) {
   }
   if (lane < p.top) {          // top <= 32 (checked by the launcher)
     p.chosen[token * p.top + lane] = my_expert;
-    p.weights[token * p.top + lane] = my_score / (picked_sum + p.weight_eps) * p.scale;
+    p.weights[token * p.top + lane] = (p.normalize ? my_score / (picked_sum + p.weight_eps) : my_score) * p.scale;
   }
 }
 
@@ -711,20 +714,31 @@ int launch_moe_gemm(const MoeGemmParams& p, bool gated, cudaStream_t stream) {
 
 template <typename TS>
 __global__ void moe_combine_kernel(const float* __restrict__ parts, const TS* __restrict__ shared,
-                                   float* __restrict__ out, int64_t total, int64_t width, int top) {
+                                   float* __restrict__ out, int64_t total, int64_t width, int top,
+                                   const int32_t* __restrict__ chosen, const float* __restrict__ pair_weights,
+                                   const void* __restrict__ x, int x_dtype, int first_identity) {
   pdl_launch_dependents();
   pdl_wait();
   const int64_t idx = blockIdx.x * (int64_t)blockDim.x + threadIdx.x;
   if (idx >= total) return;
   const int64_t token = idx / width, c = idx - token * width;
   float sum = 0.f;
-  for (int s = 0; s < top; ++s) sum += parts[(token * top + s) * width + c];
+  for (int s = 0; s < top; ++s) {
+    const int64_t pair = token * top + s;
+    if (chosen == nullptr || chosen[pair] < first_identity) {
+      sum += parts[pair * width + c];
+    } else {
+      const float v = x_dtype == kBFloat16 ? __bfloat162float(((const __nv_bfloat16*)x)[idx]) : ((const float*)x)[idx];
+      sum = fmaf(pair_weights[pair], v, sum);
+    }
+  }
   if (shared != nullptr) sum += to_float<TS>(shared[idx]);
   out[idx] = sum;
 }
 
 int launch_moe_combine(const float* parts, const void* shared, int shared_dtype, float* out, int64_t num_tokens,
-                       int64_t width, int top, cudaStream_t stream) {
+                       int64_t width, int top, const int32_t* chosen, const float* pair_weights, const void* x,
+                       int x_dtype, int first_identity, cudaStream_t stream) {
   const int64_t total = num_tokens * width;
   if (total == 0) return 0;
   const int threads = 256;
@@ -732,9 +746,11 @@ int launch_moe_combine(const float* parts, const void* shared, int shared_dtype,
   if (blocks > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
   if (shared != nullptr && shared_dtype == kBFloat16)
     return (int)launch_chain(moe_combine_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(threads), 0, stream,
-                             dim3(1, 1, 1), parts, (const __nv_bfloat16*)shared, out, total, width, top);
+                             dim3(1, 1, 1), parts, (const __nv_bfloat16*)shared, out, total, width, top, chosen,
+                             pair_weights, x, x_dtype, first_identity);
   return (int)launch_chain(moe_combine_kernel<float>, dim3((unsigned)blocks), dim3(threads), 0, stream, dim3(1, 1, 1),
-                           parts, (const float*)shared, out, total, width, top);
+                           parts, (const float*)shared, out, total, width, top, chosen, pair_weights, x, x_dtype,
+                           first_identity);
 }
 
 }  // namespace akv

@@ -101,16 +101,64 @@ class Mirrored:
         self.hidden, self.copy = hidden, copy
 
 
+class IdentityChoices:
+    """The choices of routed experts of which some hand back their input: ``chosen`` int32 and ``weights`` float32
+    [tokens, top], the input ``x`` [tokens, hidden], and ``first``, the lowest choice that is the identity.  Rows of
+    ``ExpertParts.parts`` that belong to such a choice were never written and are not read."""
+
+    def __init__(self, chosen: torch.Tensor, weights: torch.Tensor, x: torch.Tensor, first: int):
+        self.chosen, self.weights, self.x, self.first = chosen, weights, x, int(first)
+
+
 class ExpertParts:
     """A routed feed-forward's result before its sum: float32 rows ``parts`` [tokens * top, hidden] (a token's
-    ``top`` rows side by side, already weighted) and the shared expert's ``shared`` [tokens, hidden] or None.  A norm
-    that knows it adds them up in the kernel that norms them; anyone else calls :meth:`materialize`."""
+    ``top`` rows side by side, already weighted), the shared expert's ``shared`` [tokens, hidden] or None, and
+    ``identity`` (:class:`IdentityChoices`) where choices may be the identity.  A norm that knows it adds them up in
+    the kernel that norms them; anyone else calls :meth:`materialize`."""
 
-    def __init__(self, parts: torch.Tensor, shared: torch.Tensor | None, top: int):
-        self.parts, self.shared, self.top = parts, shared, int(top)
+    def __init__(self, parts: torch.Tensor, shared: torch.Tensor | None, top: int,
+                 identity: IdentityChoices | None = None):
+        self.parts, self.shared, self.top, self.identity = parts, shared, int(top), identity
 
     def materialize(self) -> torch.Tensor:
-        return moe_combine(self.parts, self.shared, top=self.top)
+        return moe_combine(self.parts, self.shared, top=self.top, identity=self.identity)
+
+
+class NormedBranch:
+    """A branch's result ``branch`` (a tensor or an :class:`ExpertParts`) that joins the stream through an RMS norm of
+    its own: ``hidden += branch / sqrt(mean(branch^2) + eps) * weight``, not done yet.  A norm that knows it
+    (``takes_normed_branch``) does both in one kernel (:func:`branch_rmsnorm`); anyone else calls :meth:`apply`."""
+
+    def __init__(self, branch, weight: torch.Tensor, eps: float):
+        if isinstance(branch, torch.Tensor) and branch.dim() == 3:       # a stack of split-K partial sums
+            branch = branch.sum(0)
+        self.branch, self.weight, self.eps = branch, weight, float(eps)
+
+    def apply(self, hidden: torch.Tensor) -> None:
+        branch_rmsnorm(hidden, self, None, 0.0, None)
+
+
+def branch_rmsnorm(hidden: torch.Tensor, pending: NormedBranch, weight: torch.Tensor | None, eps: float, out_dtype,
+                   rows: torch.Tensor | None = None, status: torch.Tensor | None = None) -> torch.Tensor | None:
+    """Add the pending branch, normed, to ``hidden`` (float32, in place), then, with ``weight``, RMS-norm the new rows:
+    ``hidden / sqrt(mean(hidden^2) + eps) * weight`` in ``out_dtype``.  With ``rows`` only those rows are made and
+    ``hidden`` is left as it is."""
+    out = None
+    if weight is not None:
+        n = hidden.shape[0] if rows is None else rows.numel()
+        out = torch.empty((n, hidden.shape[1]), dtype=out_dtype, device=hidden.device)
+    b = pending.branch
+    if isinstance(b, ExpertParts):
+        ident = b.identity
+        chosen, weights, x, first = (None, None, None, 0) if ident is None else (ident.chosen, ident.weights, ident.x,
+                                                                                ident.first)
+        ext().branch_rmsnorm(hidden, None, b.parts, b.shared, b.top, chosen, weights, x, first, pending.weight,
+                             pending.eps, weight, float(eps), out, rows, status)
+    else:
+        ext().branch_rmsnorm(hidden, b, None, None, 0, None, None, None, 0, pending.weight, pending.eps, weight,
+                             float(eps), out, rows, status)
+    _launched()
+    return out
 
 
 def branch_layernorm(hidden: torch.Tensor, branch, weight: torch.Tensor, eps: float,
@@ -119,6 +167,8 @@ def branch_layernorm(hidden: torch.Tensor, branch, weight: torch.Tensor, eps: fl
     compute dtype or float32, or an :class:`ExpertParts`).  Returns the new ``hidden`` in ``out_dtype``: a rounded
     copy, or ``hidden`` itself when ``out_dtype`` is float32."""
     copy = None if out_dtype == torch.float32 else torch.empty(hidden.shape, dtype=out_dtype, device=hidden.device)
+    if isinstance(branch, ExpertParts) and branch.identity is not None:
+        branch = branch.materialize()
     if isinstance(branch, ExpertParts):
         ext().branch_layernorm_parts(hidden, branch.parts, branch.shared, weight, copy, float(eps), branch.top)
         _launched()
@@ -415,21 +465,32 @@ def head_prep(x, slots, k_cache, v_cache, *, num_heads, num_kv_heads, head_dim, 
 
 
 def latent_prep(x, positions, slots, q_weight, kv_weight, inv_freq, cache, *, q_rank, kv_rank, rot_dim, rotary_dims,
-                eps, status=None):
-    """From one product ``x`` [tokens, query latent | key/value latent | rotated key part]: both latents through an
-    RMS norm with a plain weight, neighbouring pairs of the rotated part turned by position; the key/value latent
-    and the rotated part land side by side in the token's row of ``cache``.  Returns the query latent."""
-    q_latent = torch.empty((x.shape[0], q_rank), dtype=x.dtype, device=x.device)
+                eps, factor: float = 1.0, q_rows=None, heads: int = 0, head_dim: int = 0, has_kv: bool = True,
+                gated: bool = False, status=None):
+    """From one product ``x`` [tokens, query latent, or query heads | key/value latent | rotated key part | a gate
+    column per head | unused columns] of which the key/value columns (``has_kv``) and the gates (``gated``) may be
+    absent: the latents through an RMS norm with a plain weight, neighbouring pairs of the rotated part turned by
+    ``positions[t] * inv_freq[i]`` (cos and sin times ``factor``) while they lie in its first ``rotary_dims``; the
+    key/value latent and the rotated part land side by side in the token's row of ``cache``.  Without ``q_rank`` the
+    first columns are ``heads`` queries of ``head_dim`` unturned and ``rot_dim`` turned dims: the turned part of head h
+    goes to ``q_rows[t, h, kv_rank:]`` (``q_rows`` [tokens, heads * (kv_rank + rot_dim)], the rest of it is left
+    alone).  Returns (the query latent or None, the sigmoid of the gates float32 [tokens, heads] or None)."""
+    n = x.shape[0]
+    q_latent = torch.empty((n, q_rank), dtype=x.dtype, device=x.device) if q_rank else None
+    gate = torch.empty((n, heads), dtype=torch.float32, device=x.device) if gated else None
     ext().latent_prep(x, positions, slots, q_weight, kv_weight, inv_freq, q_latent, cache, q_rank, kv_rank, rot_dim,
-                      rotary_dims, float(eps), status)
+                      rotary_dims, float(eps), status, float(factor), q_rows, int(heads), int(head_dim), bool(has_kv),
+                      gate)
     _launched()
-    return q_latent
+    return q_latent, gate
 
 
-def rotate_pairs(x, out, positions, inv_freq, *, heads, cols, rotary_dims, in_offset, out_offset) -> None:
+def rotate_pairs(x, out, positions, inv_freq, *, heads, cols, rotary_dims, in_offset, out_offset,
+                 factor: float = 1.0) -> None:
     """``out[t, h, out_offset + c] = x[t, h, in_offset + c]`` for ``c < cols``, dims 2i and 2i + 1 of the range
-    turned by ``positions[t] * inv_freq[i]`` while they lie in the first ``rotary_dims``."""
-    ext().rotate_pairs(x, out, positions, inv_freq, heads, cols, rotary_dims, in_offset, out_offset)
+    turned by ``positions[t] * inv_freq[i]`` (cos and sin times ``factor``) while they lie in the first
+    ``rotary_dims``."""
+    ext().rotate_pairs(x, out, positions, inv_freq, heads, cols, rotary_dims, in_offset, out_offset, float(factor))
     _launched()
 
 
@@ -546,18 +607,19 @@ def moe_router_logits(x, w_router, status=None):
 MOE_SCORES = {"sigmoid": 0, "softmax": 1}
 
 
-def moe_route(logits, correction, *, top, groups, keep_groups, group_top, scale, weight_eps, score: str = "sigmoid"):
+def moe_route(logits, correction, *, top, groups, keep_groups, group_top, scale, weight_eps, score: str = "sigmoid",
+              normalize: bool = True):
     """Scores ``sigmoid(logits)``, or with ``score="softmax"`` the softmax over all experts (float32
     [tokens, experts]); choice scores are the scores plus ``correction``
     (float32 [experts] or None); experts form ``groups`` equal runs, a group's score is the sum of its ``group_top``
     largest choice scores, experts outside the ``keep_groups`` best groups cannot be chosen; the ``top`` largest
     remaining choice scores are chosen (ties: the lower index).  Returns (int32 [tokens, top], float32 [tokens, top]:
-    the chosen scores divided by their sum plus ``weight_eps``, times ``scale``)."""
+    the chosen scores divided by their sum plus ``weight_eps`` (``normalize=False``: not divided), times ``scale``)."""
     n = logits.shape[0]
     chosen = torch.empty((n, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((n, top), dtype=torch.float32, device=logits.device)
     ext().moe_route(logits, correction, chosen, weights, groups, keep_groups, group_top, float(scale), float(weight_eps),
-                    MOE_SCORES[score])
+                    MOE_SCORES[score], bool(normalize))
     _launched()
     return chosen, weights
 
@@ -598,11 +660,15 @@ def moe_down(act, w_down, order, offsets, weights, kernel: str = "auto"):
     return out
 
 
-def moe_combine(parts, shared, *, top):
+def moe_combine(parts, shared, *, top, identity: IdentityChoices | None = None):
     """``sum over a token's choices of parts[token * top + choice] (+ shared[token])`` in that order, float32
-    [tokens, hidden]."""
+    [tokens, hidden].  With ``identity`` the choices from ``identity.first`` on count as their weight times the token's
+    input instead."""
     out = torch.empty((parts.shape[0] // top, parts.shape[1]), dtype=torch.float32, device=parts.device)
-    ext().moe_combine(parts, shared, out, top)
+    if identity is None:
+        ext().moe_combine(parts, shared, out, top)
+    else:
+        ext().moe_combine(parts, shared, out, top, identity.chosen, identity.weights, identity.x, identity.first)
     _launched()
     return out
 

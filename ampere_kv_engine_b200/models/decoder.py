@@ -9,6 +9,8 @@ tokens only through the cache, and returns float32 logits for ``ctx.logit_rows``
 
 from __future__ import annotations
 
+from dataclasses import replace
+
 import torch
 
 from ..config.spec import ModelSpec
@@ -85,6 +87,13 @@ class DecoderModel:
         """One per schedule position, and behind them one for the embedding if it keeps something per request (the
         cache manager treats it as one more position without pages)."""
         specs = [self.blocks[e.layer].cache_spec() for e in self.spec.schedule]
+        # a position whose pages others read keeps them as far back as any of them looks; those name the same cache
+        for pos, entry in enumerate(self.spec.schedule):
+            if entry.cache_of is not None:
+                specs[entry.cache_of] = specs[entry.cache_of].covering(specs[pos])
+        for pos, entry in enumerate(self.spec.schedule):
+            if entry.cache_of is not None and specs[pos].stored() == specs[entry.cache_of].stored():
+                specs[pos] = replace(specs[entry.cache_of], state_shape=specs[pos].state_shape)
         own = self.embedding.cache_spec()
         if own.kind != "none":
             raise ValueError("an embedding keeps a state per request at most, no pages")

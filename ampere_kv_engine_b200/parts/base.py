@@ -13,7 +13,7 @@ here.
 
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Any, Callable
 
 import torch
@@ -84,6 +84,15 @@ class CacheSpec:
     def group_key(self) -> tuple:
         return (self.kind, self.stored(), self.window, self.chunk, self.keep_first)
 
+    def covering(self, other: "CacheSpec") -> "CacheSpec":
+        """This cache held for as long as ``other`` also needs it: what a position keeps whose pages another position
+        reads with a reach of its own.  A cache that stores something else is not covered (self is handed back)."""
+        if self.stored() != other.stored() or self.group_key() == other.group_key():
+            return self
+        if self.kind == other.kind == "window":
+            return replace(self, window=max(self.window, other.window), keep_first=max(self.keep_first, other.keep_first))
+        return replace(self, kind="full", window=None, chunk=None, keep_first=0)
+
 
 class Part:
     """Common life cycle: build from a spec, declare tensors, load them."""
@@ -130,6 +139,10 @@ class Norm(Part):
     #: return a ``LazyNorm`` for a consumer with ``takes_lazy_norm``.  A norm without it is handed ``delta=None``
     #: in that case, which means the same thing.
     takes_summed = False
+
+    #: ``forward`` takes an ``ops.NormedBranch`` as ``delta`` (a branch's result whose own norm is still to be applied
+    #: before it joins the stream).  A norm without it is handed the stream with the branch already added.
+    takes_normed_branch = False
 
 
 class PositionEncoding(Part):
@@ -274,6 +287,9 @@ class Block:
                     return lazy
             delta.launch()
             return norm.forward(hidden, None, ctx, rows=rows)
+        if isinstance(delta, ops.NormedBranch) and not norm.takes_normed_branch:
+            delta.apply(hidden)
+            delta = None
         if isinstance(delta, ops.Mirrored):
             delta = None            # the stream holds everything; the copy is of no use to a norm
         if isinstance(delta, ops.Summed):

@@ -4,13 +4,14 @@
 and 156-179).  The residual stream is float32; each branch output is handed to the next norm
 as a pending ``delta`` so that the sum and the norm are one kernel.  On decode steps the branch's
 last product may add to the stream itself and the next product apply the norm (``Summed``,
-``LazyNorm``): then no kernel stands between the two products.
+``LazyNorm``): then no kernel stands between the two products.  ``postnorm``: the norms sit on the
+branches' outputs only.  ``sandwich``: a norm before and after every branch.
 """
 
 from __future__ import annotations
 
 from ..kernels import ops
-from .base import Block, register_block
+from .base import NORMS, Block, register_block
 
 
 @register_block("prenorm")
@@ -62,6 +63,9 @@ class PostNormBlock(Block):
             if isinstance(delta, ops.PendingPhases):
                 delta.launch()
                 delta = None
+            if isinstance(delta, ops.NormedBranch):
+                delta.apply(hidden)
+                delta = None
             if delta is not None and not isinstance(delta, (ops.Summed, ops.Mirrored)):
                 raise ValueError("block kind 'postnorm' follows a block that leaves its last branch unadded; "
                                  "put a norm that adds it between them")
@@ -75,3 +79,37 @@ class PostNormBlock(Block):
                 branch = self.feed_forward.forward(x, ctx)
             x = self.feed_forward_norm.add_normed(hidden, branch, ctx)
         return hidden, ops.Mirrored(hidden, x)
+
+
+@register_block("sandwich")
+class SandwichBlock(Block):
+    """``h += norm1b(mixer(norm1(h))); h += norm2b(feed_forward(norm2(h)))``: a norm on either side of every branch (a
+    constant on the branch's normed result is a ``factor`` of its out-norm).  roles as ``prenorm`` and beside them
+    ``mixer_out_norm`` and ``feed_forward_out_norm``, which must offer ``of_branch``; without a feed-forward the layer is
+    the mixer branch alone.  A branch's result stays a pending ``ops.NormedBranch`` until the next norm: that one
+    kernel norms the branch, adds it to the float32 stream and norms the stream."""
+
+    def __init__(self, layer, **kw):
+        super().__init__(layer, **kw)
+        self.mixer_norm = self.build_role("mixer_norm")
+        self.mixer = self.build_role("mixer")
+        self.mixer_out_norm = self.build_role("mixer_out_norm", NORMS)
+        self.feed_forward = self.feed_forward_norm = self.feed_forward_out_norm = None
+        if layer.feed_forward is not None:
+            self.feed_forward_norm = self.build_role("feed_forward_norm")
+            self.feed_forward = self.build_role("feed_forward")
+            self.feed_forward_out_norm = self.build_role("feed_forward_out_norm", NORMS)
+        for norm in (self.mixer_out_norm, self.feed_forward_out_norm):
+            if norm is not None and not hasattr(norm, "of_branch"):
+                raise ValueError(f"block kind 'sandwich': norm kind {norm.spec.kind!r} cannot norm a branch's output")
+
+    def forward(self, hidden, delta, ctx, cache):
+        x = self.run_norm(self.mixer_norm, hidden, delta, ctx, consumer=self.mixer)
+        branch = self.mixer_out_norm.of_branch(self.mixer.forward(x, ctx, cache))
+        if self.feed_forward is None:
+            return hidden, branch
+        x = self.run_norm(self.feed_forward_norm, hidden, branch, ctx, consumer=self.feed_forward)
+        # a feed-forward whose result is still a sum of rows leaves the sum to the kernel that norms it
+        if getattr(self.feed_forward, "defers_sum", False):
+            return hidden, self.feed_forward_out_norm.of_branch(self.feed_forward.forward(x, ctx, defer_sum=True))
+        return hidden, self.feed_forward_out_norm.of_branch(self.feed_forward.forward(x, ctx))

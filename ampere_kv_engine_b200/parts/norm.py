@@ -18,7 +18,10 @@ from .base import Norm, ParamSpec, register_norm
 @register_norm("rmsnorm")
 class RMSNorm(Norm):
     """params: ``size`` (defaults to the hidden size), ``eps``, ``tensor`` (the weight's name under the prefix,
-    default ``weight``), ``unit_offset`` (the stored weight w is kept around zero and stands for ``1 + w``)."""
+    default ``weight``), ``unit_offset`` (the stored weight w is kept around zero and stands for ``1 + w``),
+    ``factor`` (the normed row is multiplied by this constant too: what a layer multiplies a sublayer's normed result
+    by, or a head its logits).  Beside the norm of what a branch reads (:meth:`forward`) there is the norm of what a
+    branch leaves (:meth:`of_branch`), which the next norm's kernel applies before its own."""
 
     graph_safe = True
 
@@ -29,6 +32,7 @@ class RMSNorm(Norm):
         self.eps = float(spec.params["eps"])
         self.tensor = str(spec.params.get("tensor", "weight"))
         self.unit_offset = bool(spec.params.get("unit_offset", False))
+        self.factor = float(spec.params.get("factor", 1.0))
         self.weight: torch.Tensor | None = None
 
     def param_specs(self):
@@ -37,12 +41,21 @@ class RMSNorm(Norm):
     def load(self, tensors):
         # the factor the kernels multiply by: the stored weight, or one more than it (formed once, in float32)
         self.weight = tensors[self.tensor] + 1.0 if self.unit_offset else tensors[self.tensor]
+        if self.factor != 1.0:
+            self.weight = self.weight * self.factor
 
     takes_summed = True
     takes_pending = True
+    takes_normed_branch = True
+
+    def of_branch(self, branch):
+        """The norm of a branch's result, to be added to the stream by whoever reads the stream next."""
+        return ops.NormedBranch(branch, self.weight, self.eps)
 
     def forward(self, hidden, delta, ctx, rows=None, lazy=False):
         status = getattr(ctx, "status", None)
+        if isinstance(delta, ops.NormedBranch):
+            return ops.branch_rmsnorm(hidden, delta, self.weight, self.eps, self.dtype, rows=rows, status=status)
         if isinstance(delta, ops.PendingPhases):
             if lazy and rows is None and self.size == hidden.shape[1] and self.weight.data_ptr() % 16 == 0:
                 return ops.StreamNorm(delta, self.weight, self.eps, self.dtype)

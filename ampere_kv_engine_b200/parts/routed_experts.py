@@ -6,7 +6,9 @@
     groups  : the experts form ``groups`` equal runs of neighbours; a group's score is the sum of its ``group_top``
               largest c; only experts of the ``keep_groups`` best groups can be chosen
     chosen  = the ``top`` allowed experts with the largest c
-    w_e     = s_e / (sum of the chosen s + weight_eps) * route_scale
+    w_e     = s_e / (sum of the chosen s + weight_eps) * route_scale   (``normalize=False``: s_e * route_scale)
+    choices from ``experts`` on (``identity`` of them) are the identity: w_e x, no matrices; the router, the scores,
+              the correction and the groups count them like experts
     expert  : g = min(W_gate x, limit); u = clamp(W_up x, -limit, limit); W_down (g * sigmoid(slope * g) * (u + 1))
               (``activation="silu"``: plain W_down (silu(W_gate x) * W_up x), no clamp)
     y       = sum_e w_e expert_e(x)  +  shared(x)
@@ -29,7 +31,9 @@ from .base import FeedForward, ParamSpec, register_feed_forward
 @register_feed_forward("routed_experts")
 class RoutedExperts(FeedForward):
     """params: ``experts``, ``top``, ``groups`` and ``keep_groups`` (default 1 / 1: no groups), ``group_top``
-    (default 2; 1: a group is scored by its best expert), ``route_scale``, ``weight_eps``, ``score`` (``"sigmoid"`` or
+    (default 2; 1: a group is scored by its best expert), ``identity`` (choices beyond the experts that hand back their
+    input, default 0), ``normalize`` (default True: the chosen scores are divided by their sum), ``route_scale``,
+    ``weight_eps``, ``score`` (``"sigmoid"`` or
     ``"softmax"``), ``correction`` (bool, default True: a learned per-expert offset of the choice scores),
     ``activation`` (``"clamped_swish"``, the default, with ``limit`` and ``swish_slope``; or ``"silu"``),
     ``intermediate_size`` of an expert, ``shared`` (None, or ``{"intermediate_size", "limit"}``), ``names`` (``expert`` with ``{}`` for
@@ -46,14 +50,19 @@ class RoutedExperts(FeedForward):
         super().__init__(spec, **kw)
         p = spec.params
         self.experts, self.top = int(p["experts"]), int(p["top"])
+        self.identity = int(p.get("identity") or 0)
+        if self.identity < 0:
+            raise ValueError("routed_experts: identity must not be negative")
+        self.choices = self.experts + self.identity       # what the router scores
+        self.normalize = bool(p.get("normalize", True))
         self.groups, self.keep_groups = int(p.get("groups") or 1), int(p.get("keep_groups") or 1)
         self.group_top = int(p.get("group_top", 2))
-        if self.experts <= 0 or self.experts % self.groups or not 0 < self.keep_groups <= self.groups:
-            raise ValueError(f"routed_experts: {self.experts} experts do not form {self.groups} equal groups of which "
+        if self.experts <= 0 or self.choices % self.groups or not 0 < self.keep_groups <= self.groups:
+            raise ValueError(f"routed_experts: {self.choices} experts do not form {self.groups} equal groups of which "
                              f"{self.keep_groups} are kept")
-        if not 0 < self.top <= self.keep_groups * (self.experts // self.groups):
+        if not 0 < self.top <= self.keep_groups * (self.choices // self.groups):
             raise ValueError(f"routed_experts: top {self.top} is more than the kept groups hold")
-        if self.experts > ops.MOE_MAX_EXPERTS or self.top > ops.MOE_MAX_TOP:
+        if self.choices > ops.MOE_MAX_EXPERTS or self.top > ops.MOE_MAX_TOP:
             raise ValueError(f"routed_experts: the kernels take up to {ops.MOE_MAX_EXPERTS} experts and a top of "
                              f"{ops.MOE_MAX_TOP}")
         self.score = str(p.get("score", "sigmoid"))
@@ -87,9 +96,9 @@ class RoutedExperts(FeedForward):
             specs[self._expert(e, "gate")] = ParamSpec((f, h))
             specs[self._expert(e, "up")] = ParamSpec((f, h))
             specs[self._expert(e, "down")] = ParamSpec((h, f))
-        specs[n["router"]] = ParamSpec((self.experts, h))
+        specs[n["router"]] = ParamSpec((self.choices, h))
         if self.has_correction:
-            specs[n["correction"]] = ParamSpec((self.experts,), kind="vector", init="around_zero")
+            specs[n["correction"]] = ParamSpec((self.choices,), kind="vector", init="around_zero")
         if self.shared_size:
             specs[f"{n['shared']}.{n['gate']}"] = ParamSpec((self.shared_size, h))
             specs[f"{n['shared']}.{n['up']}"] = ParamSpec((self.shared_size, h))
@@ -114,8 +123,11 @@ class RoutedExperts(FeedForward):
         logits = ops.moe_router_logits(x, self.w_router, status=status)
         chosen, weights = ops.moe_route(logits, self.correction, top=self.top, groups=self.groups,
                                         keep_groups=self.keep_groups, group_top=self.group_top,
-                                        scale=self.route_scale, weight_eps=self.weight_eps, score=self.score)
-        order, offsets = ops.moe_sort(chosen, self.experts)
+                                        scale=self.route_scale, weight_eps=self.weight_eps, score=self.score,
+                                        normalize=self.normalize)
+        order, offsets = ops.moe_sort(chosen, self.choices)
+        if self.identity:
+            offsets = offsets[:self.experts + 1]       # the identity choices' pairs sort behind the experts' runs
         act = ops.moe_gate_up(x, self.w_gate_up, order, offsets, top=self.top, limit=self.limit,
                               slope=self.swish_slope, up_offset=self.up_offset)
         parts = ops.moe_down(act, self.w_down, order, offsets, weights)
@@ -128,5 +140,6 @@ class RoutedExperts(FeedForward):
                 both = ops.linear(x, self.shared_gate_up, status=status)
                 shared = ops.linear(ops.glu(both, "clamped_swish", 0, self.shared_limit, self.swish_slope),
                                     self.shared_down, status=status)
-        result = ops.ExpertParts(parts, shared, self.top)
+        identity = ops.IdentityChoices(chosen, weights, x, self.experts) if self.identity else None
+        result = ops.ExpertParts(parts, shared, self.top, identity)
         return result if defer_sum else result.materialize()

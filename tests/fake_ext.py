@@ -266,12 +266,12 @@ class FakeExt:
             v_cache[s // page_size, :, s % page_size] = v[keep].to(v_cache.dtype)
 
     @staticmethod
-    def _turn_pairs(t, positions, inv_freq, rotary_dims):
+    def _turn_pairs(t, positions, inv_freq, rotary_dims, factor=1.0):
         if rotary_dims == 0:
             return t
         ang = positions.float()[:, None] * inv_freq[None, :]
         shape = [t.shape[0]] + [1] * (t.dim() - 2) + [rotary_dims // 2]
-        cos, sin = ang.cos().view(shape), ang.sin().view(shape)
+        cos, sin = ang.cos().view(shape) * factor, ang.sin().view(shape) * factor
         out = t.clone()
         u, v = t[..., 0:rotary_dims:2], t[..., 1:rotary_dims:2]
         out[..., 0:rotary_dims:2] = u * cos - v * sin
@@ -279,24 +279,47 @@ class FakeExt:
         return out
 
     def latent_prep(self, x, positions, slots, q_weight, kv_weight, inv_freq, q_latent, cache, q_rank, kv_rank,
-                    rot_dim, rotary_dims, eps, status=None):
+                    rot_dim, rotary_dims, eps, status=None, factor=1.0, q_rows=None, heads=0, head_dim=0, has_kv=True,
+                    gate=None):
         xf = x.float()
-        a, b, r = xf[:, :q_rank], xf[:, q_rank:q_rank + kv_rank], xf[:, q_rank + kv_rank:]
-        q_latent.copy_((a * torch.rsqrt(a.square().mean(-1, keepdim=True) + eps) * q_weight).to(q_latent.dtype))
+        n = x.shape[0]
+        first = q_rank or heads * (head_dim + rot_dim)
+        a, b, r = xf[:, :first], xf[:, first:first + kv_rank], xf[:, first + kv_rank:first + kv_rank + rot_dim]
+        if q_rank:
+            q_latent.copy_((a * torch.rsqrt(a.square().mean(-1, keepdim=True) + eps) * q_weight).to(q_latent.dtype))
+        else:
+            turned = self._turn_pairs(a.view(n, heads, -1)[:, :, head_dim:], positions, inv_freq, rotary_dims, factor)
+            q_rows.view(n, heads, -1)[:, :, kv_rank:] = turned.to(q_rows.dtype)
+        if gate is not None:
+            off = first + (kv_rank + rot_dim if has_kv else 0)
+            gate.copy_(torch.sigmoid(xf[:, off:off + heads]))
         if cache is None or slots is None:
             return
         c = b * torch.rsqrt(b.square().mean(-1, keepdim=True) + eps) * kv_weight
-        row = torch.cat((c, self._turn_pairs(r, positions, inv_freq, rotary_dims)), dim=-1)
+        row = torch.cat((c, self._turn_pairs(r, positions, inv_freq, rotary_dims, factor)), dim=-1)
         page_size = cache.shape[2]
         keep = slots >= 0
         s = slots[keep].long()
         cache[s // page_size, 0, s % page_size, :row.shape[1]] = row[keep].to(cache.dtype)
 
-    def rotate_pairs(self, x, out, positions, inv_freq, heads, cols, rotary_dims, in_offset, out_offset):
+    def rotate_pairs(self, x, out, positions, inv_freq, heads, cols, rotary_dims, in_offset, out_offset, factor=1.0):
         n = x.shape[0]
         part = x.view(n, heads, -1)[:, :, in_offset:in_offset + cols].float()
         out.view(n, heads, -1)[:, :, out_offset:out_offset + cols] = \
-            self._turn_pairs(part, positions, inv_freq, rotary_dims).to(out.dtype)
+            self._turn_pairs(part, positions, inv_freq, rotary_dims, factor).to(out.dtype)
+
+    def branch_rmsnorm(self, hidden, branch, parts, shared, top, chosen, pair_weights, x, first_identity, weight, eps,
+                       next_weight, next_eps, out, rows=None, status=None):
+        if branch is None:
+            branch = torch.empty_like(hidden)
+            self.moe_combine(parts, shared, branch, top, chosen, pair_weights, x, first_identity)
+        b = branch.float()
+        new = hidden + b * torch.rsqrt(b.square().mean(-1, keepdim=True) + eps) * weight
+        if rows is None:
+            hidden.copy_(new)
+        if out is not None:
+            y = new if rows is None else new[rows.long()]
+            out.copy_((y * torch.rsqrt(y.square().mean(-1, keepdim=True) + next_eps) * next_weight).to(out.dtype))
 
     def activation(self, x, out, kind):
         z = x.float()
@@ -583,7 +606,7 @@ class FakeExt:
     # ------------------------------------------------------------------ routed experts
 
     def moe_route(self, logits, correction, chosen, weights, groups, keep_groups, group_top, scale, weight_eps,
-                  score_kind=0):
+                  score_kind=0, normalize=True):
         n, E = logits.shape
         top = chosen.shape[1]
         s = torch.sigmoid(logits.float()) if score_kind == 0 else torch.softmax(logits.float(), dim=-1)
@@ -599,7 +622,7 @@ class FakeExt:
         ids = torch.sort(masked, dim=-1, descending=True, stable=True).indices[:, :top]
         picked = s.gather(1, ids)
         chosen.copy_(ids.to(torch.int32))
-        weights.copy_(picked / (picked.sum(-1, keepdim=True) + weight_eps) * scale)
+        weights.copy_((picked / (picked.sum(-1, keepdim=True) + weight_eps) if normalize else picked) * scale)
 
     def moe_router(self, x, w, logits):
         logits.copy_(x.float() @ w.float().T)
@@ -631,6 +654,10 @@ class FakeExt:
                 continue
             out[rows] = (act[off[e]:off[e + 1]].float() @ w_down[e].float().T) * flat[rows][:, None]
 
-    def moe_combine(self, parts, shared, out, top):
-        total = parts.view(-1, top, parts.shape[1]).sum(1)
+    def moe_combine(self, parts, shared, out, top, chosen=None, pair_weights=None, x=None, first_identity=0):
+        rows = parts.view(-1, top, parts.shape[1])
+        if chosen is not None:       # rows of identity choices were never written
+            same = chosen.view(-1, top, 1) >= first_identity
+            rows = torch.where(same, pair_weights.view(-1, top, 1) * x.float()[:, None, :], rows)
+        total = rows.sum(1)
         out.copy_(total if shared is None else total + shared.float())

@@ -86,7 +86,7 @@ def test_latent_prep_and_pair_rotation(dtype, q_rank, kv_rank, rot_dim, dims, he
     inv_freq = (base ** (-2.0 * i / dims)).float().cuda()
     slots = torch.randperm(pages * page_size, generator=g, device="cuda")[:n].to(torch.int32)
     cache = torch.zeros((pages, 1, page_size, kv_rank + rot_dim), device="cuda", dtype=dtype)
-    q_latent = ops.latent_prep(x, positions, slots, wq, wkv, inv_freq, cache, q_rank=q_rank, kv_rank=kv_rank,
+    q_latent, _ = ops.latent_prep(x, positions, slots, wq, wkv, inv_freq, cache, q_rank=q_rank, kv_rank=kv_rank,
                                rot_dim=rot_dim, rotary_dims=dims, eps=eps)
     xd, pos = x.double().cpu(), positions.cpu().long()
     tol = dict(TOL[dtype])
