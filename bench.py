@@ -1,6 +1,6 @@
 """Benchmark of the engine on one B200: decode tokens per second at the Qwen3-8B shape.
 
-    python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--impl reference] [--shape 8b|14b|32b|sukalorn|zifuzen|renadra|zavizen]
+    python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--impl reference] [--shape 8b|14b|32b|sukalorn|zifuzen|renadra|zavizen|ligirax]
 
 Prints ONE JSON line.  A "step" is one decode step of the whole batch through the engine's own step
 function (every kernel of the model and the token choice); ``value`` is batch / step time, timed with CUDA
@@ -14,6 +14,8 @@ cache) with the copy bandwidth.  Weights are random (seeded), token ids syntheti
 Renadra's kernels alone beside the like kernels of the other designs.
 ``--shape zavizen`` sets four Zavizen layers beside Renadra layers of equal size, and Zavizen's kernels alone beside the
 like kernels of the other designs.
+``--shape ligirax`` sets four Ligirax layers beside Zifuzen attention layers with experts of equal size, Ligirax's mixers
+alone beside Sukalorn's latent mixers of equal size, and Ligirax's kernels alone beside the like kernels of those.
 ``--shape sukalorn`` prints a line of its own: prefill and decode of four Sukalorn layers at two sizes beside Qwen3
 layers of equal size, and the attention kernels alone.
 Between timed steps nothing is flushed: every step streams the whole model (16 GB at full depth) through
@@ -569,6 +571,52 @@ def zavizen_config(z: dict, layers: int) -> dict:
                         "mlp": {"kind": "dense", "ff": z["ff"]}} for i in range(layers)]}
 
 
+# Ligirax at sizes that resemble a real model's layers: four layers of latent attention behind a window (the third reads
+# the second's latents) with routed experts of which some choices are the identity.  Its closest designs: Zifuzen for the
+# feed-forward (attention with as many key/value heads as in the sizes above, the same experts and top, softmax scores
+# apart), Sukalorn for the mixer (latent attention over the same heads, widths and rank, behind a query latent, over all
+# keys); the mixers are measured in layers without a feed-forward.
+LIGIRAX_SIZES = {
+    "2k": dict(width=2048, heads=16, kv_heads=4, dim=128, rot_dim=64, q_rank=768, kv_rank=512, window=1024, experts=32,
+               identity=8, top=6, expert_ff=768),
+    "4k": dict(width=4096, heads=32, kv_heads=8, dim=128, rot_dim=64, q_rank=1536, kv_rank=512, window=1024, experts=64,
+               identity=16, top=6, expert_ff=1024),
+}
+
+
+def ligirax_config(z: dict, layers: int, feed_forward: bool = True) -> dict:
+    mixer = {"heads": z["heads"], "dim": z["dim"], "rot_dim": z["rot_dim"], "vdim": z["dim"], "kv_rank": z["kv_rank"],
+             "scale": (z["dim"] + z["rot_dim"]) ** -0.5, "mask": {"size": z["window"]},
+             "rot": {"base": 10000.0, "dims": z["rot_dim"],
+                     "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"], "limit": 7.0},
+           "router": {"experts": z["experts"], "identity": z["identity"], "top": z["top"]}}
+    out = [{"type": "latent_attention", "mixer": json.loads(json.dumps(mixer)),
+            "mlp": json.loads(json.dumps(moe)) if feed_forward else None} for _ in range(layers)]
+    if layers > 2:
+        out[2]["mixer"]["kv_from"] = 1
+    return {"architecture": "Ligirax", "vocab": SUKALORN_VOCAB, "width": z["width"], "norm": {"eps": 1e-6},
+            "residual_mult": 0.5, "logit_scale": 2.0, "layers": out}
+
+
+def ligirax_like_experts(z: dict, layers: int) -> dict:
+    attention = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"],
+                 "scale": z["dim"] ** -0.5}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"], "limit": 7.0},
+           "router": {"experts": z["experts"], "top": z["top"], "scale": 1.0}}
+    return {"architecture": "Zifuzen", "vocab": SUKALORN_VOCAB, "width": z["width"], "max_positions": CONTEXT,
+            "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "logit_softcap": None,
+            "layers": [{"type": "attention", "mixer": dict(attention), "mlp": json.loads(json.dumps(moe))}
+                       for _ in range(layers)]}
+
+
+def ligirax_like_mixers(z: dict, layers: int) -> dict:
+    latent = sukalorn_config(dict(z, block=z["window"], ff=1), 2)["layers"][1]["mixer"]
+    return {"architecture": "Sukalorn", "vocab": SUKALORN_VOCAB, "width": z["width"], "norm": {"eps": 1e-6},
+            "layers": [{"type": "latent_attention", "mixer": json.loads(json.dumps(latent)), "mlp": None}
+                       for _ in range(layers)]}
+
+
 def zifuzen_dense_like(z: dict, layers: int) -> dict:
     attention = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"],
                  "scale": z["dim"] ** -0.5}
@@ -1084,7 +1132,135 @@ def sukalorn_shape(args, design: str = "sukalorn") -> int:
                    moved=moved)
         return out
 
+    def ligirax_kernels_alone(z: dict) -> dict:
+        """The kernels that came with the Ligirax design by themselves at this size, each beside the like kernel of
+        another design: attention over shared rows behind a window with gates beside the same over all keys without
+        (Sukalorn), the latent mixer's preparation with direct queries beside the one with a query latent and the pair
+        rotation behind it, the norm of a branch and of the stream in one pass beside the branch LayerNorm (Zifuzen) and
+        the residual add + RMS norm, both with a stored branch and with experts' rows, the routing, and the grouped
+        products with identity choices beside the same with none."""
+        out = {}
+        heads, dim, R, rank, W = z["heads"], z["dim"], z["rot_dim"], z["kv_rank"], z["width"]
+        E, I, top, F, page, window = z["experts"], z["identity"], z["top"], z["expert_ff"], args.page_size, z["window"]
+        row = rank + R
+        bf = dict(dtype=torch.bfloat16, device=device)
+        g = torch.Generator(device=device).manual_seed(4)
+        dev = lambda v: torch.tensor(v, dtype=torch.int32, device=device)
+
+        def record(key, fn, *, flops=0.0, moved=0.0):
+            for _ in range(3):
+                fn()
+            ms = timed(fn, 5, flush_l2=True)
+            entry = {"ms": round(ms, 4)}
+            if flops:
+                entry["tflops"] = round(flops / (ms / 1000) / 1e12, 2)
+                entry["frac_of_bf16_peak"] = round(flops / (ms / 1000) / 1e12 / peaks["bf16_tflops"], 4)
+            if moved:
+                entry["gbs"] = round(moved / (ms / 1000) / 1e9, 1)
+                entry["frac_of_hbm"] = round(moved / (ms / 1000) / 1e9 / peaks["hbm_gbs"], 4)
+            out[key] = entry
+
+        for name, seq_q, q_tile in (("prompt", [(PREFILL_TOKENS, PREFILL_TOKENS)], ops.ATTENTION_Q_TILE),
+                                    ("decode", [(PROMPT_LEN, 1)] * batch, 1)):
+            lay, pages, tokens = layout(seq_q, q_tile)
+            rand = lambda *shape: torch.randn(shape, generator=g, **bf)
+            rows, q_row = rand(pages, 1, page, row), rand(tokens, heads * row)
+            gate = torch.rand((tokens, heads), device=device, generator=g)
+            for case, reach, gates in (("latent_window_attention", window, gate), ("like_sukalorn_latent_attention", 0, None)):
+                pairs = sum(min(c - n + i + 1, reach or c) for c, n in seq_q for i in range(n))
+                keys = sum(min(c, reach or c) for c, _ in seq_q)
+                splits = ops.choose_splits_shared_rows(lay["num_tiles"], 1, q_tile * heads, min(max(c for c, _ in seq_q), reach or 1 << 30))
+                record(f"{name}_{case}", lambda: ops.scored_attention(
+                    q_row, rows, rows, num_splits=splits, num_heads=heads, num_kv_heads=1, v_dim=rank, scale=0.07,
+                    window=reach, gate=gates, **lay), flops=2.0 * heads * (row + rank) * pairs, moved=2.0 * row * keys)
+                out[f"{name}_{case}"]["splits"] = splits
+            # the preparation: what it reads of the product, what it writes
+            positions = dev([c - n + i for c, n in seq_q for i in range(n)])
+            slots = dev(list(range(tokens)))
+            freq = torch.rand((R // 2,), device=device, generator=g)
+            weight = torch.ones((rank,), device=device)
+            x = rand(tokens, heads * (dim + R) + row + heads)
+            prep = dict(kv_rank=rank, rot_dim=R, rotary_dims=R, eps=1e-6)
+            record(f"{name}_latent_prep_direct_queries", lambda: ops.latent_prep(
+                x, positions, slots, None, weight, freq, rows, q_rank=0, factor=1.1, q_rows=q_row, heads=heads,
+                head_dim=dim, gated=True, **prep), moved=tokens * (4.0 * heads * R + 4.0 * row + 6.0 * heads))
+            qr = z["q_rank"]
+            xl, ql, q_weight = rand(tokens, qr + row), rand(tokens, heads * (dim + R)), torch.ones((qr,), device=device)
+            record(f"{name}_like_latent_prep_query_latent", lambda: ops.latent_prep(
+                xl, positions, slots, q_weight, weight, freq, rows, q_rank=qr, **prep), moved=tokens * (4.0 * qr + 4.0 * row))
+            record(f"{name}_like_rotate_pairs", lambda: ops.rotate_pairs(
+                ql, q_row, positions, freq, heads=heads, cols=R, rotary_dims=R, in_offset=dim, out_offset=rank),
+                moved=tokens * 4.0 * heads * R)
+            # a stored branch: hidden read and written, the branch read, the next input written
+            hidden = torch.randn((tokens, W), device=device, generator=g)
+            branch, ones = rand(tokens, W), torch.ones((W,), device=device)
+            record(f"{name}_branch_rmsnorm", lambda: ops.branch_rmsnorm(
+                hidden, ops.NormedBranch(branch, ones, 1e-6), ones, 1e-6, torch.bfloat16), moved=tokens * W * 12.0)
+            record(f"{name}_like_branch_layernorm", lambda: ops.branch_layernorm(hidden, branch, ones, 1e-6, torch.bfloat16),
+                   moved=tokens * W * 12.0)
+            record(f"{name}_like_add_rmsnorm", lambda: ops.add_rmsnorm(hidden, branch, ones, 1e-6, torch.bfloat16),
+                   moved=tokens * W * 12.0)
+            # the routed feed-forward
+            logits = torch.randn((tokens, E + I), device=device, generator=g)
+            correction = torch.zeros((E + I,), device=device)
+            route = lambda score, norm, z_, corr: ops.moe_route(
+                z_, corr, top=top, groups=1, keep_groups=1, group_top=1, scale=1.0, weight_eps=1e-20, score=score, normalize=norm)
+            record(f"{name}_moe_route", lambda: route("softmax", False, logits, correction), moved=4.0 * tokens * (E + I))
+            plain_logits = logits[:, :E].contiguous()
+            record(f"{name}_like_moe_route", lambda: route("sigmoid", True, plain_logits, correction[:E].contiguous()),
+                   moved=4.0 * tokens * E)
+            w_gu = (torch.randn((E, 2 * F, W), device=device, generator=g) * 0.02).to(torch.bfloat16)
+            w_d = (torch.randn((E, W, F), device=device, generator=g) * 0.02).to(torch.bfloat16)
+            for tag, chosen, weights, choices in (("", *route("softmax", False, logits, correction), E + I),
+                                                  ("like_", *route("sigmoid", True, plain_logits, None), E)):
+                record(f"{name}_{tag}moe_sort", lambda: ops.moe_sort(chosen, choices), moved=8.0 * tokens * top)
+                order, offsets = ops.moe_sort(chosen, choices)
+                offsets = offsets[:E + 1]
+                rows_used, used = int(offsets[-1]), int((offsets[1:] > offsets[:-1]).sum())
+                record(f"{name}_{tag}moe_gate_up", lambda: ops.moe_gate_up(branch, w_gu, order, offsets, top=top, limit=7.0,
+                                                                          slope=1.702),
+                       flops=4.0 * rows_used * F * W, moved=2.0 * used * 2 * F * W)
+                act = ops.moe_gate_up(branch, w_gu, order, offsets, top=top, limit=7.0, slope=1.702)
+                record(f"{name}_{tag}moe_down", lambda: ops.moe_down(act, w_d, order, offsets, weights),
+                       flops=2.0 * rows_used * F * W, moved=2.0 * used * F * W)
+                parts = ops.moe_down(act, w_d, order, offsets, weights)
+                for entry in ("moe_gate_up", "moe_down"):
+                    out[f"{name}_{tag}{entry}"]["rows"] = rows_used
+                ident = ops.IdentityChoices(chosen, weights, branch, E) if not tag else None
+                pieces = ops.ExpertParts(parts, None, top, ident)
+                if not tag:
+                    record(f"{name}_branch_rmsnorm_experts", lambda: ops.branch_rmsnorm(
+                        hidden, ops.NormedBranch(pieces, ones, 1e-6), ones, 1e-6, torch.bfloat16),
+                        moved=W * (4.0 * rows_used + tokens * 12.0))
+                else:
+                    record(f"{name}_like_branch_layernorm_experts", lambda: ops.branch_layernorm(
+                        hidden, pieces, ones, 1e-6, torch.bfloat16), moved=W * (4.0 * rows_used + tokens * 10.0))
+        return out
+
     sizes = {}
+    if design == "ligirax":
+        with ClockSampler() as clocks:
+            for name, z in LIGIRAX_SIZES.items():
+                sizes[name] = {"ligirax": measure(ligirax_config(z, layers)),
+                               "zifuzen_attention_experts": measure(ligirax_like_experts(z, layers)),
+                               "ligirax_mixers": measure(ligirax_config(z, layers, feed_forward=False)),
+                               "sukalorn_latent_mixers": measure(ligirax_like_mixers(z, layers)),
+                               "kernels": ligirax_kernels_alone(z)}
+        head = sizes["4k"]["ligirax"]
+        line = {"metric": "decode tok/s at batch 8 of four Ligirax layers (width 4,096, B200); prefill, a smaller size, "
+                          "Zifuzen attention layers with experts of equal size, both designs' latent mixers alone and "
+                          "Ligirax's kernels alone, each beside the like kernel of another design, alongside",
+                "value": head["decode_tok_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
+                "warmup": args.warmup, "ms_per_step": head["decode_ms"], "higher_is_better": True, "dtype": "bf16",
+                "data": "synthetic (seeded uniform token ids, seeded random weights)",
+                "config": {"model": "Ligirax", "layers": layers, "sizes": LIGIRAX_SIZES, "vocab": SUKALORN_VOCAB,
+                           "global_batch": batch, "prompt_len": PROMPT_LEN, "prefill_tokens": PREFILL_TOKENS,
+                           "page_size": args.page_size, "l2": "whole steps: inputs larger than L2; kernels alone: L2 "
+                           "flushed (a 256 MB write) before every timed launch", "peaks": peaks["source"]},
+                "gpu_launches": head["launches_per_decode_step"] * args.steps, "sizes": sizes,
+                "clocks": clocks.summary()}
+        print(json.dumps(line))
+        return 0
     if design == "zavizen":
         with ClockSampler() as clocks:
             for name, z in RENADRA_SIZES.items():
@@ -1175,19 +1351,20 @@ def main() -> int:
     parser.add_argument("--warmup", type=int, default=8)
     parser.add_argument("--impl", choices=("ours", "reference"), default="ours")
     parser.add_argument("--page-size", type=int, default=PAGE_SIZE, help="tokens per cache page (a power of two, 16 or more)")
-    parser.add_argument("--shape", choices=sorted(SHAPES) + ["renadra", "sukalorn", "zavizen", "zifuzen"], default="8b",
+    parser.add_argument("--shape", choices=sorted(SHAPES) + ["ligirax", "renadra", "sukalorn", "zavizen", "zifuzen"], default="8b",
                         help="8b: the headline benchmark; 14b: a mixed scheduler load of 64 requests; 32b: long-context "
                              "decode at batch 16; sukalorn: prefill and decode of the Sukalorn design at two layer "
                              "sizes beside Qwen3 layers of equal size; zifuzen: the same for the Zifuzen design; renadra: the Renadra design beside "
                              "Zifuzen layers of equal size; zavizen: the Zavizen design beside Renadra layers of equal "
-                             "size (each prints its own one line)")
+                             "size; ligirax: the Ligirax design beside Zifuzen's experts and Sukalorn's latent mixer "
+                             "(each prints its own one line)")
     parser.add_argument("--layers", type=int, default=None,
                         help="run fewer layers of the same sizes (reported in config beside the full count)")
     parser.add_argument("--batch", type=int, default=8)
     parser.add_argument("--no-points", action="store_true", help="skip the batch-1 and batch-64 decode points")
     args = parser.parse_args()
 
-    if args.shape in ("renadra", "sukalorn", "zavizen", "zifuzen"):
+    if args.shape in ("ligirax", "renadra", "sukalorn", "zavizen", "zifuzen"):
         if args.impl == "reference":
             print(json.dumps({"impl": "reference", "unavailable": "the reference arm runs the 8b shape only"}))
             return 0

@@ -102,13 +102,11 @@ def mixture(h: torch.Tensor, w: dict, mlp: dict, margins: list | None = None) ->
     if margins is not None:
         margins.append(lead)
     out = torch.zeros_like(h)
-    for t in range(h.shape[0]):
-        for e, weight in zip(chosen[t].tolist(), weights[t]):
-            if e >= real:
-                out[t] += weight * h[t]
-            else:
-                out[t] += weight * clamped_expert(h[t], w[f"e{e}.gate"], w[f"e{e}.up"], w[f"e{e}.down"],
+    for e in sorted(set(chosen.flatten().tolist())):
+        t, place = (chosen == e).nonzero(as_tuple=True)          # the tokens that chose e
+        y = h[t] if e >= real else clamped_expert(h[t], w[f"e{e}.gate"], w[f"e{e}.up"], w[f"e{e}.down"],
                                                   mlp["expert"]["limit"])
+        out[t] += weights[t, place][:, None] * y
     return out
 
 
