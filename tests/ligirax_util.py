@@ -110,6 +110,8 @@ def model_folder(name: str, seed: int = 3) -> str:
     t = load_file(path)
     narrow = (72.0 / cfg.width) ** 0.5                # products of about the same size at every width
     t["embed"] = t["embed"] * 20.0
+    # of both signs: a tied head would otherwise answer every token with itself
+    t["final.norm"] = torch.randn(cfg.width, generator=torch.Generator().manual_seed(seed + 100))
     for i, lay in enumerate(cfg.layers):
         m = lay.mixer
         # unrotated and rotated scores with a spread of a few units before the scale
