@@ -939,3 +939,175 @@ class LigiraxConfig:
         if self.eos_token_id:
             out["eos_token_id"] = list(self.eos_token_id)
         return out
+
+
+@dataclass(frozen=True)
+class GosizenLayer:
+    """One layer of a Gosizen model as config.json gives it: ``type`` names the mixer, ``mixer`` holds its sizes and
+    constants, ``mlp`` the feed-forward's (None: the layer has none)."""
+
+    type: str
+    mixer: dict
+    mlp: dict | None
+
+    MIXERS = ("latent_attention", "parallel")
+
+
+@dataclass(frozen=True)
+class GosizenConfig:
+    """config.json of the ``Gosizen`` decoder: ``vocab``, ``width``, ``norm.eps``, ``token_side.dim`` (the width of a
+    layer's token input; absent: none), ``logit_softcap`` (absent: none), a list of layers and an optional ``loop``
+    (``start``, ``stop``, ``times``: the run of layers [start, stop) is walked ``times`` times on one set of weights, a
+    projection of the stream beside the embedding's output before every walk).  A layer names its mixer
+    (``latent_attention``: ``heads``, ``dim``, ``rot_dim``, ``vdim``, ``q_rank``, ``kv_rank``, ``scale``, ``rot``,
+    ``mask.size`` (a window); ``parallel``: a ``left`` attention with ``heads``, ``kv_heads``, ``dim``, ``vdim``,
+    ``conv``, ``scale``, ``rot`` (with an optional ``scaling``: ``factor``, ``original``, ``low``, ``high``), ``mask.size``
+    (a block of positions) beside a ``right`` delta rule with ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``conv`` and, for
+    random weights alone, ``decay_rank`` and ``gate_rank``, which a checkpoint's own shapes say otherwise; ``left_scale``,
+    ``right_scale``) and its feed-forward (``kind`` ``dense`` with ``ff``, or ``moe`` with ``expert.ff`` and ``router``
+    (``experts``, ``top``); or null).  Every size and constant is read from here or from a tensor's shape."""
+
+    vocab: int
+    width: int
+    norm_eps: float
+    layers: tuple[GosizenLayer, ...]
+    loop: dict | None = None
+    side_dim: int | None = None
+    logit_softcap: float | None = None
+    max_position_embeddings: int = 1 << 20
+    eos_token_id: tuple[int, ...] = ()
+    architectures: tuple[str, ...] = ("Gosizen",)
+
+    ARCHITECTURE = "Gosizen"
+
+    @property
+    def vocab_size(self) -> int:
+        return self.vocab
+
+    @staticmethod
+    def _check_rot(m: dict, where: str, dim: int, name: str) -> None:
+        rot = _section(m, "rot", where)
+        where_r = where + "rot: "
+        dims = _sized(rot, "dims", where_r)
+        if _number(rot, "base", where_r) <= 1:
+            raise ConfigError(f"config.json: {where_r}'base' must be above 1")
+        if dims % 2 or dims > dim:
+            raise ConfigError(f"config.json: {where_r}'dims' must be even and at most '{name}' ({dim}), got {dims}")
+        if rot.get("scaling") is not None:
+            s = _section(rot, "scaling", where_r)
+            for key in ("factor", "original", "low", "high"):
+                if _number(s, key, where_r + "scaling: ") <= 0:
+                    raise ConfigError(f"config.json: {where_r}scaling: '{key}' must be positive")
+            if s["low"] >= s["high"]:
+                raise ConfigError(f"config.json: {where_r}scaling: 'low' ({s['low']}) must be below 'high' ({s['high']})")
+
+    @staticmethod
+    def _check_heads(m: dict, where: str) -> None:
+        for key in ("heads", "kv_heads", "dim", "vdim", "conv"):
+            _sized(m, key, where)
+        if m["heads"] % m["kv_heads"]:
+            raise ConfigError(f"config.json: {where}'heads' ({m['heads']}) must be a multiple of 'kv_heads' "
+                              f"({m['kv_heads']})")
+
+    @classmethod
+    def _check_mixer(cls, kind: str, m: dict, where: str) -> None:
+        if kind == "latent_attention":
+            for key in ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank"):
+                _sized(m, key, where)
+            _number(m, "scale", where)
+            cls._check_rot(m, where, m["rot_dim"], "rot_dim")
+            if m.get("mask") is not None:
+                _sized(_section(m, "mask", where), "size", where + "mask: ")
+            return
+        left, right = _section(m, "left", where), _section(m, "right", where)
+        cls._check_heads(left, where + "left: ")
+        _number(left, "scale", where + "left: ")
+        cls._check_rot(left, where + "left: ", left["dim"], "dim")
+        if left.get("mask") is not None:
+            _sized(_section(left, "mask", where + "left: "), "size", where + "left: mask: ")
+        cls._check_heads(right, where + "right: ")
+        for key in ("decay_rank", "gate_rank"):
+            if right.get(key) is not None:
+                _sized(right, key, where + "right: ")
+        for key in ("left_scale", "right_scale"):
+            _number(m, key, where)
+
+    @staticmethod
+    def _check_mlp(mlp: dict, where: str) -> None:
+        kind = mlp.get("kind", "dense")
+        if kind == "dense":
+            _sized(mlp, "ff", where)
+            return
+        if kind != "moe":
+            raise ConfigError(f"config.json: {where}'kind' must be 'dense' or 'moe', got {kind!r}")
+        _sized(_section(mlp, "expert", where), "ff", where + "expert: ")
+        router, where_r = _section(mlp, "router", where), where + "router: "
+        experts, top = _sized(router, "experts", where_r), _sized(router, "top", where_r)
+        if top > experts:
+            raise ConfigError(f"config.json: {where_r}'top' ({top}) is more than the {experts} experts there are")
+
+    @classmethod
+    def from_dict(cls, d: dict[str, Any]) -> "GosizenConfig":
+        layers_raw = d.get("layers")
+        if not isinstance(layers_raw, (list, tuple)) or not layers_raw:
+            raise ConfigError("config.json: key 'layers' must be a non-empty list")
+        layers = []
+        for i, entry in enumerate(layers_raw):
+            where = f"layers[{i}]: "
+            if not isinstance(entry, dict) or entry.get("type") not in GosizenLayer.MIXERS:
+                raise ConfigError(f"config.json: {where}'type' must be one of {list(GosizenLayer.MIXERS)}, "
+                                  f"got {entry.get('type') if isinstance(entry, dict) else entry!r}")
+            mixer = _section(entry, "mixer", where)
+            cls._check_mixer(entry["type"], mixer, where + "mixer: ")
+            mlp = entry.get("mlp")
+            if mlp is not None:
+                if not isinstance(mlp, dict):
+                    raise ConfigError(f"config.json: {where}'mlp' must be an object or null")
+                cls._check_mlp(mlp, where + "mlp: ")
+            layers.append(GosizenLayer(entry["type"], copy.deepcopy(mixer), None if mlp is None else copy.deepcopy(mlp)))
+        loop = d.get("loop")
+        if loop is not None:
+            loop = _section(d, "loop", "")
+            times = _sized(loop, "times", "loop: ")
+            start, stop = loop.get("start"), loop.get("stop")
+            if not all(isinstance(v, int) and not isinstance(v, bool) for v in (start, stop)) or \
+                    not 0 <= start < stop <= len(layers):
+                raise ConfigError(f"config.json: loop: 'start' and 'stop' must satisfy 0 <= start < stop <= "
+                                  f"{len(layers)}, got {start!r} and {stop!r}")
+            loop = {"start": start, "stop": stop, "times": times}
+        side = None
+        if d.get("token_side") is not None:
+            side = _sized(_section(d, "token_side", ""), "dim", "token_side: ")
+        eos = d.get("eos_token_id")
+        eos = () if eos is None else ((eos,) if isinstance(eos, int) else tuple(eos))
+        cap = d.get("logit_softcap")
+        cfg = cls(
+            vocab=_sized(d, "vocab", ""),
+            width=_sized(d, "width", ""),
+            norm_eps=_number(_section(d, "norm", ""), "eps", "norm: "),
+            layers=tuple(layers),
+            loop=loop,
+            side_dim=side,
+            logit_softcap=None if cap is None else _number(d, "logit_softcap", ""),
+            max_position_embeddings=_optional(d, "max_position_embeddings", int, 1 << 20),
+            eos_token_id=eos,
+        )
+        if cfg.norm_eps <= 0:
+            raise ConfigError("config.json: norm: 'eps' must be positive")
+        if cfg.logit_softcap is not None and cfg.logit_softcap <= 0:
+            raise ConfigError("config.json: 'logit_softcap' must be positive (or null for none)")
+        return cfg
+
+    def to_dict(self) -> dict[str, Any]:
+        out = {"architecture": self.ARCHITECTURE, "vocab": self.vocab, "width": self.width,
+               "norm": {"eps": self.norm_eps}, "logit_softcap": self.logit_softcap,
+               "token_side": None if self.side_dim is None else {"dim": self.side_dim},
+               "layers": [{"type": l.type, "mixer": copy.deepcopy(l.mixer),
+                           "mlp": None if l.mlp is None else copy.deepcopy(l.mlp)} for l in self.layers]}
+        if self.loop is not None:
+            out["loop"] = dict(self.loop)
+        if self.max_position_embeddings != 1 << 20:
+            out["max_position_embeddings"] = self.max_position_embeddings
+        if self.eos_token_id:
+            out["eos_token_id"] = list(self.eos_token_id)
+        return out

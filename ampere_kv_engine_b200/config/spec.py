@@ -74,12 +74,15 @@ class ScheduleEntry:
     otherwise).  ``cache_of`` names an earlier position of the schedule whose cache this
     position reads instead of writing one of its own.  ``add_embedding``: the embedding's output (the
     residual stream as it was before the first position) is added to the stream right before this position runs,
-    as a model does that sends the stream through a run of layers again.
+    as a model does that sends the stream through a run of layers again.  ``begins_walk``: this position is the first of
+    a pass through a run of layers, the ``begins_walk``-th (from 0); the model's ``walk_entry`` acts on the stream right
+    before it.
     """
 
     layer: int
     cache_of: int | None = None
     add_embedding: bool = False
+    begins_walk: int | None = None
 
 
 @dataclass(frozen=True)
@@ -99,6 +102,8 @@ class ModelSpec:
     #: copies of the residual stream per token (0: the one plain stream).  With copies the decoder hands the blocks
     #: [tokens, streams, width], all copies equal to the embedding's row at first, and norms their sum at the end.
     streams: int = 0
+    #: a stream update that stands before every position that ``begins_walk``
+    walk_entry: PartSpec | None = None
 
     def validate(self) -> None:
         if not self.schedule:
@@ -107,6 +112,9 @@ class ModelSpec:
             raise ValueError("model spec: streams must not be negative")
         if self.streams and any(e.add_embedding for e in self.schedule):
             raise ValueError("model spec: adding the embedding again is not defined for a stream in several copies")
+        walks = [e.begins_walk for e in self.schedule if e.begins_walk is not None]
+        if walks and (self.walk_entry is None or self.streams):
+            raise ValueError("model spec: a position that begins a pass needs a walk_entry (and one plain stream)")
         for pos, entry in enumerate(self.schedule):
             if not 0 <= entry.layer < len(self.layers):
                 raise ValueError(f"model spec: schedule position {pos} names layer {entry.layer}, "

@@ -89,6 +89,7 @@ struct TcParams {
   int sigmoid = 0;
   const float* head_bias = nullptr;
   float out_scale = 1.f;
+  const float* sink = nullptr;
 };
 
 // Byte offset of (key k, 16-byte chunk c of the head) inside one stage's K or V area.  The area is laid out
@@ -666,6 +667,18 @@ attention_decode_coop_kernel(const __grid_constant__ CUtensorMap k_map, const __
       if (live[1]) head_bias[1] = tp.head_bias[kvh * G + row_b] * kLog2e;
     }
 
+    // a sink: the first split's walk starts as if a key of that score and of value zero had come first (every warp
+    // holds the maximum, one lane of the CTA counts the one)
+    if (kScored && tp.sink != nullptr && split == 0) {
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        if (live[r]) {
+          m[r] = tp.sink[kvh * G + (r ? row_b : row_a)] * kLog2e;
+          l[r] = (warp == 0 && (lane & 3) == 0) ? 1.f : 0.f;
+        }
+      }
+    }
+
     for (int b = 0; b < num_blocks; ++b) {
       const int s = b % STAGES;
       uint8_t* stage = smem + s * Layout::kStage;
@@ -952,7 +965,7 @@ int launch_coop_scored(const ScoredAttentionParams& sp, int box_rows, const CUte
     configured = true;
   }
   TcParams tp{p, box_rows, sp.softcap, sp.slopes, sp.chunk, sp.gate,
-              sp.keep_first, sp.sigmoid_weights, sp.head_bias, sp.out_scale};
+              sp.keep_first, sp.sigmoid_weights, sp.head_bias, sp.out_scale, sp.sink};
   const dim3 grid((unsigned)p.num_tiles, (unsigned)p.num_kv_heads, (unsigned)p.num_splits);
   const dim3 cluster(1, 1, CLUSTER ? (unsigned)p.num_splits : 1u);
   return (int)launch_chain(kernel, grid, dim3((kCoopWarps + 1) * 32), smem, stream, cluster, k_map, v_map, tp);

@@ -132,6 +132,7 @@ struct FaParams {
   int sigmoid = 0;
   const float* head_bias = nullptr;
   float out_scale = 1.f;
+  const float* sink = nullptr;      // the denominator also counts exp(sink[h])
 };
 
 // Shared memory: Q [2 halves][128 rows][128 B] | K/V ring: per stage K [2][64][128 B], V [2][64][128 B] |
@@ -429,6 +430,11 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
     // inside the sigmoid, in log2 units
     const float head_bias = (sigmoid && fp.head_bias != nullptr) ? fp.head_bias[kvh * G + head_local] * kLog2e : 0.f;
     float m_ref = -CUDART_INF_F, l = 0.f;
+    // a sink: the walk starts as if a key of that score and of value zero had come first
+    if (kScored && fp.sink != nullptr && live) {
+      m_ref = fp.sink[kvh * G + head_local] * kLog2e;
+      l = 1.f;
+    }
 
     for (int b = 0; b < num_blocks; ++b) {
       const int s = b % kStagesKV;
@@ -1100,7 +1106,7 @@ int launch_attention_tcgen05_scored(const ScoredAttentionParams& sp, cudaStream_
       !cache_map(p.v_cache, rows, box_rows, &v_map))
     return (int)cudaErrorInvalidValue;
   FaParams fp{p, tq, subtiles, box_rows, sp.softcap, sp.slopes, sp.chunk, sp.gate,
-              sp.keep_first, sp.sigmoid_weights, sp.head_bias, sp.out_scale};
+              sp.keep_first, sp.sigmoid_weights, sp.head_bias, sp.out_scale, sp.sink};
   fp.p.num_splits = 1;
   const dim3 grid((unsigned)(p.num_tiles * subtiles), (unsigned)p.num_kv_heads, 1u);
   // two CTAs per SM with two K/V stages each when there are more CTAs than SMs, else one with four stages

@@ -212,7 +212,7 @@ struct TokenOperand {
   const void* x = nullptr;
   akv::GemmNormedX normed = {};
   bool is_normed = false;
-  int64_t tokens = 0, k = 0;
+  int64_t tokens = 0, k = 0, x_stride = 0;      // x_stride: elements between two rows of x (0: k)
   const Tensor* anchor = nullptr;     // device and stream
 };
 
@@ -224,9 +224,11 @@ TokenOperand token_operand(const OptTensor& x, const OptTensor& nx_hidden, const
   TokenOperand t;
   if (x.has_value()) {
     AKV_CHECK(!nx_hidden.has_value(), "give x or the residual stream to norm, not both");
-    check_cuda(*x, "x");
-    AKV_CHECK(x->scalar_type() == at::kBFloat16 && x->dim() == 2 && x->size(1) == w.size(1),
+    AKV_CHECK(x->is_cuda() && x->scalar_type() == at::kBFloat16 && x->dim() == 2 && x->size(1) == w.size(1),
               "x must be bfloat16 [tokens, k] for w [features, k]");
+    AKV_CHECK(x->is_contiguous() || (x->stride(1) == 1 && x->stride(0) >= x->size(1) && x->stride(0) % 8 == 0),
+              "x must be contiguous, or columns of a wider matrix whose rows start on 16-byte boundaries");
+    t.x_stride = x->is_contiguous() ? 0 : x->stride(0);
     AKV_CHECK(reinterpret_cast<uintptr_t>(x->data_ptr()) % 16 == 0, "x must be 16-byte aligned");
     t.x = x->data_ptr();
     t.tokens = x->size(0);
@@ -275,9 +277,10 @@ void small_m_gemm(const OptTensor& x, const Tensor& w, Tensor& out, int64_t spli
   const TokenOperand t = token_operand(x, nx_hidden, nx_ssq, nx_weight, nx_eps, w);
   check_cuda(out, "out");
   AKV_CHECK(out.device() == w.device(), "out and w must be on the same device");
-  AKV_CHECK(activation >= -1 && activation <= 2 &&
+  AKV_CHECK(activation >= -1 && activation <= akv::kActLast &&
                 (activation < 0 || (!gated && out.dim() == 2 && out.scalar_type() == at::kBFloat16)),
-            "an activation (0 relu squared, 1 tanh GELU, 2 SiLU) goes with the plain product and a bfloat16 out");
+            "an activation (0 relu squared, 1 tanh GELU, 2 SiLU, 3 GELU with erf) goes with the plain product and a "
+            "bfloat16 out");
   void* out_ptr = nullptr;
   float* parts_ptr = nullptr;
   int out_code = 0;
@@ -308,6 +311,7 @@ void small_m_gemm(const OptTensor& x, const Tensor& w, Tensor& out, int64_t spli
   f.normed_x = t.is_normed;
   f.normed = t.normed;
   f.activation = (int)activation;
+  f.x_stride = t.x_stride;
   c10::cuda::CUDAGuard guard(w.device());
   check_launch(akv::launch_small_m_gemm(t.x, w.data_ptr(), out_ptr, out_code, parts_ptr, t.tokens, w.size(0), t.k,
                                         (int)splits, &f, status_ptr(status), stream_of(*t.anchor)),
@@ -330,6 +334,7 @@ void small_m_gemm_residual(const Tensor& x, const Tensor& w, Tensor& hidden, Ten
   check_cluster_splits(splits, t.k);
   akv::GemmFusion f;
   f.epilogue = akv::kEpilogueResidual;
+  f.x_stride = t.x_stride;
   f.residual.hidden = hidden.data_ptr<float>();
   f.residual.ssq = ssq.data_ptr<float>();
   c10::cuda::CUDAGuard guard(w.device());
@@ -405,6 +410,7 @@ void small_m_gemm_qkv(const OptTensor& x, const Tensor& w, Tensor& q_out, const 
   e.num_kv_heads = (int)num_kv_heads;
   e.eps = (float)eps;
   akv::GemmFusion f;
+  f.x_stride = t.x_stride;
   f.epilogue = akv::kEpilogueQkv;
   f.qkv = e;
   f.normed_x = t.is_normed;
@@ -721,7 +727,7 @@ void scored_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
                       int64_t q_tile, int64_t num_splits, int64_t num_heads, int64_t num_kv_heads, int64_t v_dim,
                       int64_t window, int64_t chunk, double scale, double softcap, const OptTensor& slopes,
                       const OptTensor& gate, const OptTensor& status, int64_t kernel, int64_t keep_first,
-                      bool sigmoid_weights, const OptTensor& head_bias, double out_scale) {
+                      bool sigmoid_weights, const OptTensor& head_bias, double out_scale, const OptTensor& sink) {
   check_cuda(q, "q");
   check_cuda(out, "out");
   check_same(q, out, "q", "out");
@@ -805,6 +811,11 @@ void scored_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
     sp.head_bias = head_bias->data_ptr<float>();
   }
   sp.out_scale = (float)out_scale;
+  if (sink.has_value()) {
+    AKV_CHECK(!sigmoid_weights, "scored_attention: a sink goes with a softmax");
+    check_f32(*sink, "sink", num_heads);
+    sp.sink = sink->data_ptr<float>();
+  }
   c10::cuda::CUDAGuard guard(q.device());
   check_launch(akv::launch_scored_attention(sp, stream_of(q)), "scored_attention");
 }
@@ -985,7 +996,8 @@ void activation(const Tensor& in, Tensor& out, int64_t kind) {
   check_cuda(out, "out");
   check_same(in, out, "in", "out");
   AKV_CHECK(in.numel() == out.numel(), "in and out must have the same number of elements");
-  AKV_CHECK(kind >= 0 && kind <= 2, "activation: kind must be 0 (relu squared), 1 (tanh GELU) or 2 (SiLU)");
+  AKV_CHECK(kind >= 0 && kind <= akv::kActLast,
+            "activation: kind must be 0 (relu squared), 1 (tanh GELU), 2 (SiLU) or 3 (GELU with erf)");
   c10::cuda::CUDAGuard guard(in.device());
   check_launch(akv::launch_activation(in.data_ptr(), out.data_ptr(), in.numel(), (int)kind, dtype_code(in, "in"),
                                       stream_of(in)),
@@ -1184,8 +1196,10 @@ void softcap(Tensor& logits, double cap) {
   check_launch(akv::launch_softcap(logits.data_ptr<float>(), logits.numel(), (float)cap, stream_of(logits)), "softcap");
 }
 
+// x [tokens, at least x_off + q | k | v columns]; without further tensors the rest of x is [gate | beta | step].
 akv::DeltaParams delta_params(const Tensor& x, const Tensor& state, const Tensor& cu_q, const Tensor& state_slots,
-                              int64_t num_heads, int64_t num_kv_heads, int64_t head_dim, int64_t v_dim, int64_t taps) {
+                              int64_t num_heads, int64_t num_kv_heads, int64_t head_dim, int64_t v_dim, int64_t taps,
+                              int64_t x_off, bool whole) {
   check_cuda(x, "x");
   AKV_CHECK(num_heads > 0 && num_kv_heads > 0 && num_heads % num_kv_heads == 0 && head_dim > 0 && v_dim > 0,
             "delta rule: sizes must be positive and heads a multiple of the q/k heads");
@@ -1194,12 +1208,15 @@ akv::DeltaParams delta_params(const Tensor& x, const Tensor& state, const Tensor
   AKV_CHECK(taps >= 1 && taps <= akv::kDeltaMaxTaps, "delta rule: taps must be between 1 and ", (int64_t)akv::kDeltaMaxTaps);
   const int64_t channels = 2 * num_kv_heads * head_dim + num_heads * v_dim;
   const int64_t width = channels + num_heads * v_dim + 2 * num_heads;
-  AKV_CHECK(x.dim() == 2 && x.size(1) == width, "x must be [tokens, ", width, "]: q, k, v, gate, beta, step");
+  if (whole) AKV_CHECK(x.dim() == 2 && x.size(1) == width && x_off == 0, "x must be [tokens, ", width, "]: q, k, v, gate, beta, step");
+  else AKV_CHECK(x.dim() == 2 && x_off >= 0 && x_off + channels <= x.size(1), "x must hold ", channels, " q, k and v columns from x_off on");
   const int64_t memory = akv::delta_memory_floats((int)num_heads, (int)head_dim, (int)v_dim);
   const int64_t floats = (memory + (taps - 1) * channels + 3) / 4 * 4;
-  check_cuda(state, "state");
-  AKV_CHECK(state.scalar_type() == at::kFloat && state.dim() == 2 && state.size(1) == floats && state.device() == x.device(),
-            "state must be float32 [slots, ", floats, "]");
+  AKV_CHECK(state.is_cuda() && state.scalar_type() == at::kFloat && state.dim() == 2 && state.size(1) == floats &&
+                state.stride(1) == 1 && state.device() == x.device(),
+            "state must be float32 [slots, ", floats, "] (rows may lie further apart)");
+  AKV_CHECK(state.size(0) <= 1 || (state.stride(0) >= floats && state.stride(0) % 4 == 0),
+            "the state's rows must start on 16-byte boundaries");
   check_i32(cu_q, "cu_q", 1);
   const int64_t num_seqs = cu_q.numel() - 1;
   check_i32(state_slots, "state_slots", num_seqs);
@@ -1209,7 +1226,7 @@ akv::DeltaParams delta_params(const Tensor& x, const Tensor& state, const Tensor
   p.cu_q = cu_q.data_ptr<int>();
   p.state_slots = state_slots.data_ptr<int>();
   p.num_tokens = x.size(0);
-  p.state_stride = state.size(1);
+  p.state_stride = state.stride(0);
   p.memory = memory;
   p.num_seqs = (int)num_seqs;
   p.num_slots = (int)state.size(0);
@@ -1219,19 +1236,51 @@ akv::DeltaParams delta_params(const Tensor& x, const Tensor& state, const Tensor
   p.v_dim = (int)v_dim;
   p.taps = (int)taps;
   p.dtype = dtype_code(x, "x");
+  p.x_stride = x.size(1);
+  p.x_off = (int)x_off;
+  p.beta_off = (int)(channels + num_heads * v_dim);
+  p.coef_stride = 2 * num_heads;
+  p.gates = x.data_ptr();
+  p.gate_stride = x.size(1);
+  p.gate_off = (int)channels;
+  p.gate_dtype = p.dtype;
+  p.steps = x.data_ptr();
+  p.step_stride = x.size(1);
+  p.step_off = p.beta_off + (int)num_heads;
+  p.step_dtype = p.dtype;
+  p.out_stride = num_heads * v_dim;
+  p.factor = 1.f;
   return p;
 }
 
+// steps: [tokens, at least the step columns from step_off], a tensor of its own (float32 or bfloat16), or none: in x.
 void delta_prep(const Tensor& x, const Tensor& conv, const Tensor& rate_log, const Tensor& step_bias, const Tensor& state,
                 const Tensor& cu_q, const Tensor& state_slots, Tensor& qkv, Tensor& coef, int64_t num_heads,
-                int64_t num_kv_heads, int64_t head_dim, int64_t v_dim, int64_t taps, double unit_eps) {
-  akv::DeltaParams p = delta_params(x, state, cu_q, state_slots, num_heads, num_kv_heads, head_dim, v_dim, taps);
+                int64_t num_kv_heads, int64_t head_dim, int64_t v_dim, int64_t taps, double unit_eps,
+                const OptTensor& steps, int64_t step_off, bool channel_decay, int64_t x_off, int64_t beta_off) {
+  akv::DeltaParams p = delta_params(x, state, cu_q, state_slots, num_heads, num_kv_heads, head_dim, v_dim, taps, x_off,
+                                    !steps.has_value());
   const int64_t channels = 2 * num_kv_heads * head_dim + num_heads * v_dim;
+  const int64_t per_token = channel_decay ? num_heads * head_dim : num_heads;
+  AKV_CHECK(!channel_decay || steps.has_value(), "delta_prep: decays per channel come from a tensor of their own");
+  if (steps.has_value()) {
+    check_cuda(*steps, "steps");
+    AKV_CHECK(steps->dim() == 2 && steps->size(0) == p.num_tokens && step_off >= 0 && step_off + per_token <= steps->size(1) &&
+                  steps->device() == x.device(), "steps must be [tokens, at least ", per_token, " columns from step_off]");
+    AKV_CHECK(beta_off >= 0 && beta_off + num_heads <= x.size(1), "delta_prep: the beta columns must lie inside x");
+    p.steps = steps->data_ptr();
+    p.step_stride = steps->size(1);
+    p.step_off = (int)step_off;
+    p.step_dtype = dtype_code(*steps, "steps");
+    p.beta_off = (int)beta_off;
+  }
+  p.channel_decay = channel_decay ? 1 : 0;
+  p.coef_stride = num_heads + per_token;
   check_f32(conv, "conv", channels * taps);
   check_f32(rate_log, "rate_log", num_heads);
-  check_f32(step_bias, "step_bias", num_heads);
+  check_f32(step_bias, "step_bias", per_token);
   check_f32(qkv, "qkv", p.num_tokens * channels);
-  check_f32(coef, "coef", p.num_tokens * 2 * num_heads);
+  check_f32(coef, "coef", p.num_tokens * p.coef_stride);
   p.conv = conv.data_ptr<float>();
   p.rate_log = rate_log.data_ptr<float>();
   p.step_bias = step_bias.data_ptr<float>();
@@ -1242,23 +1291,46 @@ void delta_prep(const Tensor& x, const Tensor& conv, const Tensor& rate_log, con
   check_launch(akv::launch_delta_prep(p, stream_of(x)), "delta_prep");
 }
 
+// gates: [tokens, at least heads * v_dim columns from gate_off], a tensor of its own, or none: in x.  out: [tokens, at
+// least heads * v_dim columns from out_off].
 void delta_scan(const Tensor& qkv, const Tensor& coef, const Tensor& x, const Tensor& norm_weight, Tensor& state,
                 const Tensor& cu_q, const Tensor& state_slots, Tensor& scratch, Tensor& out, int64_t num_heads,
-                int64_t num_kv_heads, int64_t head_dim, int64_t v_dim, int64_t taps, double norm_eps) {
-  akv::DeltaParams p = delta_params(x, state, cu_q, state_slots, num_heads, num_kv_heads, head_dim, v_dim, taps);
+                int64_t num_kv_heads, int64_t head_dim, int64_t v_dim, int64_t taps, double norm_eps,
+                const OptTensor& gates, int64_t gate_off, int64_t gate_kind, bool channel_decay, int64_t x_off,
+                int64_t out_off, double factor) {
+  akv::DeltaParams p = delta_params(x, state, cu_q, state_slots, num_heads, num_kv_heads, head_dim, v_dim, taps, x_off,
+                                    !gates.has_value());
   const int64_t channels = 2 * num_kv_heads * head_dim + num_heads * v_dim;
+  p.channel_decay = channel_decay ? 1 : 0;
+  p.coef_stride = num_heads + (channel_decay ? num_heads * head_dim : num_heads);
   check_f32(qkv, "qkv", p.num_tokens * channels);
-  check_f32(coef, "coef", p.num_tokens * 2 * num_heads);
+  check_f32(coef, "coef", p.num_tokens * p.coef_stride);
   check_f32(norm_weight, "norm_weight", v_dim);
   check_f32(scratch, "scratch", p.num_tokens * num_heads * v_dim);
   check_cuda(out, "out");
   check_same(out, x, "out", "x");
-  AKV_CHECK(out.numel() == p.num_tokens * num_heads * v_dim, "out must be [tokens, heads * v_dim]");
+  AKV_CHECK(out.dim() == 2 && out.size(0) == p.num_tokens && out_off >= 0 && out_off + num_heads * v_dim <= out.size(1),
+            "out must be [tokens, at least heads * v_dim columns from out_off]");
+  AKV_CHECK(gate_kind == 0 || gate_kind == 1, "delta_scan: gate_kind 0 (SiLU) or 1 (sigmoid)");
+  if (gates.has_value()) {
+    check_cuda(*gates, "gates");
+    AKV_CHECK(gates->dim() == 2 && gates->size(0) == p.num_tokens && gate_off >= 0 &&
+                  gate_off + num_heads * v_dim <= gates->size(1) && gates->device() == x.device(),
+              "gates must be [tokens, at least heads * v_dim columns from gate_off]");
+    p.gates = gates->data_ptr();
+    p.gate_stride = gates->size(1);
+    p.gate_off = (int)gate_off;
+    p.gate_dtype = dtype_code(*gates, "gates");
+  }
+  p.gate_kind = (int)gate_kind;
   p.qkv = qkv.data_ptr<float>();
   p.coef = coef.data_ptr<float>();
   p.norm_weight = norm_weight.data_ptr<float>();
   p.scratch = scratch.data_ptr<float>();
   p.out = out.data_ptr();
+  p.out_stride = out.size(1);
+  p.out_off = (int)out_off;
+  p.factor = (float)factor;
   p.norm_eps = (float)norm_eps;
   c10::cuda::CUDAGuard guard(x.device());
   check_launch(akv::launch_delta_scan(p, stream_of(x)), "delta_scan");
@@ -1713,7 +1785,7 @@ void ssm_prep(const Tensor& x, const Tensor& conv, const OptTensor& conv_bias, c
 
 // The last taps - 1 inputs of `channels` convolved columns of x, per sequence, into the state slot behind tail_off.
 void conv_tail(const Tensor& x, Tensor& state, int64_t tail_off, const Tensor& cu_q, const Tensor& state_slots,
-               int64_t conv_off, int64_t channels, int64_t taps) {
+               int64_t conv_off, int64_t channels, int64_t taps, const OptTensor& bias) {
   check_cuda(x, "x");
   AKV_CHECK(x.dim() == 2 && channels >= 1 && taps >= 1 && taps <= akv::kConvMaxTaps && conv_off >= 0 &&
                 conv_off + channels <= x.size(1), "conv_tail: the channels must lie inside x; 1 to ",
@@ -1726,6 +1798,10 @@ void conv_tail(const Tensor& x, Tensor& state, int64_t tail_off, const Tensor& c
   check_i32(state_slots, "state_slots", seqs);
   akv::ConvTailParams p{};
   p.x = x.data_ptr();
+  if (bias.has_value()) {
+    check_f32(*bias, "bias", channels);
+    p.bias = bias->data_ptr<float>();
+  }
   p.x_stride = x.size(1);
   p.conv_off = (int)conv_off;
   p.channels = (int)channels;
@@ -1742,9 +1818,205 @@ void conv_tail(const Tensor& x, Tensor& state, int64_t tail_off, const Tensor& c
   check_launch(akv::launch_conv_tail(p, stream_of(x)), "conv_tail");
 }
 
+// q, k and v of a product (from column x_off) plus their biases through short convolutions, q and k turned, k and v to
+// the cache (see launchers.h).
+void conv_rotary_prep(const Tensor& x, int64_t x_off, const OptTensor& bias, const Tensor& conv, const OptTensor& state,
+                      int64_t tail_off, const Tensor& cu_q, const Tensor& state_slots, const Tensor& positions,
+                      const Tensor& slots, const Tensor& freq, Tensor& q_out, Tensor& k_cache, Tensor& v_cache,
+                      int64_t num_heads, int64_t num_kv_heads, int64_t head_dim, int64_t v_dim, int64_t taps,
+                      int64_t rotary_dims, int64_t layout, double factor, bool keep_tail, const OptTensor& status) {
+  check_cuda(x, "x");
+  check_cuda(q_out, "q_out");
+  check_same(x, q_out, "x", "q_out");
+  AKV_CHECK(num_heads > 0 && num_kv_heads > 0 && head_dim > 0 && v_dim > 0, "conv_rotary_prep: sizes must be positive");
+  AKV_CHECK(rotary_dims >= 0 && rotary_dims % 2 == 0 && rotary_dims <= head_dim && rotary_dims <= 1024 &&
+                (layout == 0 || layout == 1),
+            "conv_rotary_prep: rotary_dims must be even and at most the head's width; layout 0 or 1");
+  AKV_CHECK(taps >= 1 && taps <= akv::kConvMaxTaps, "conv_rotary_prep: 1 to ", (int64_t)akv::kConvMaxTaps, " taps");
+  const int64_t channels = (num_heads + num_kv_heads) * head_dim + num_kv_heads * v_dim, n = x.size(0);
+  AKV_CHECK(x.dim() == 2 && x_off >= 0 && x_off + channels <= x.size(1), "x must hold ", channels,
+            " q, k and v columns from x_off on");
+  check_f32(conv, "conv", channels * taps);
+  check_i32(cu_q, "cu_q");
+  const int64_t seqs = cu_q.numel() - 1;
+  AKV_CHECK(seqs >= 1, "cu_q must hold at least one sequence");
+  check_i32(state_slots, "state_slots", seqs);
+  check_i32(positions, "positions", n);
+  check_i32(slots, "slots", n);
+  check_f32(freq, "freq", rotary_dims / 2);
+  AKV_CHECK(q_out.numel() == n * num_heads * head_dim, "q_out must be [tokens, heads * head_dim]");
+  check_pages(k_cache, "k_cache", num_kv_heads, head_dim, x);
+  check_pages(v_cache, "v_cache", num_kv_heads, v_dim, x);
+  AKV_CHECK(k_cache.size(0) == v_cache.size(0) && k_cache.size(2) == v_cache.size(2),
+            "k_cache and v_cache must have the same pages and page size");
+  AKV_CHECK(!keep_tail || n == seqs, "conv_rotary_prep: the tail is kept where every sequence has one token");
+  akv::ConvPrepParams p{};
+  p.x = static_cast<const char*>(x.data_ptr()) + x_off * x.element_size();
+  p.x_stride = x.size(1);
+  if (bias.has_value()) {
+    check_f32(*bias, "bias", channels);
+    p.bias = bias->data_ptr<float>();
+  }
+  p.conv = conv.data_ptr<float>();
+  if (taps > 1) {
+    AKV_CHECK(state.has_value() && state->is_cuda() && state->scalar_type() == at::kFloat && state->dim() == 2 &&
+                  state->stride(1) == 1 && tail_off >= 0 && tail_off + (taps - 1) * channels <= state->size(1),
+              "state must be float32 [slots, floats] with room for the convolutions' inputs behind tail_off");
+    p.state = state->data_ptr<float>();
+    p.state_stride = state->stride(0);
+    p.tail_off = tail_off;
+    p.num_slots = (int)state->size(0);
+  }
+  p.cu_q = cu_q.data_ptr<int>();
+  p.state_slots = state_slots.data_ptr<int>();
+  p.positions = positions.data_ptr<int>();
+  p.slots = slots.data_ptr<int>();
+  p.freq = freq.data_ptr<float>();
+  p.q_out = q_out.data_ptr();
+  p.k_cache = k_cache.data_ptr();
+  p.v_cache = v_cache.data_ptr();
+  p.num_tokens = n;
+  p.num_pages = k_cache.size(0);
+  p.k_row_stride = k_cache.size(3);
+  p.v_row_stride = v_cache.size(3);
+  p.channels = (int)channels;
+  p.taps = (int)taps;
+  p.num_seqs = (int)seqs;
+  p.num_heads = (int)num_heads;
+  p.num_kv_heads = (int)num_kv_heads;
+  p.head_dim = (int)head_dim;
+  p.v_dim = (int)v_dim;
+  p.page_size = (int)k_cache.size(2);
+  p.rotary_dims = (int)rotary_dims;
+  p.layout = (int)layout;
+  p.factor = (float)factor;
+  p.keep_tail = (keep_tail && taps > 1) ? 1 : 0;
+  p.dtype = dtype_code(x, "x");
+  p.status = status_ptr(status);
+  c10::cuda::CUDAGuard guard(x.device());
+  check_launch(akv::launch_conv_rotary_prep(p, stream_of(x)), "conv_rotary_prep");
+}
+
+// out[:, out_off + c] = in[:, c] * sigmoid(x[:, gate_off + c]) * factor
+void gate_columns(const Tensor& in, const Tensor& x, int64_t gate_off, Tensor& out, int64_t out_off, double factor) {
+  check_cuda(in, "in");
+  check_cuda(x, "x");
+  check_cuda(out, "out");
+  check_same(in, x, "in", "x");
+  check_same(in, out, "in", "out");
+  AKV_CHECK(in.dim() == 2 && x.dim() == 2 && out.dim() == 2 && x.size(0) == in.size(0) && out.size(0) == in.size(0) &&
+                gate_off >= 0 && gate_off + in.size(1) <= x.size(1) && out_off >= 0 && out_off + in.size(1) <= out.size(1),
+            "gate_columns: the gate columns must lie inside x, the results inside out");
+  c10::cuda::CUDAGuard guard(in.device());
+  check_launch(akv::launch_gate_columns(in.data_ptr(), static_cast<const char*>(x.data_ptr()) + gate_off * x.element_size(),
+                                        static_cast<char*>(out.data_ptr()) + out_off * out.element_size(), in.size(0),
+                                        (int)in.size(1), x.size(1), out.size(1), (float)factor, dtype_code(in, "in"),
+                                        stream_of(in)), "gate_columns");
+}
+
+// out[:, out_off + c] = activation(in[:, off + c]) for c < width
+void activation_columns(const Tensor& in, int64_t off, int64_t width, int64_t kind, Tensor& out, int64_t out_off) {
+  check_cuda(in, "in");
+  check_cuda(out, "out");
+  check_same(in, out, "in", "out");
+  AKV_CHECK(in.dim() == 2 && out.dim() == 2 && in.size(0) == out.size(0) && off >= 0 && width >= 0 &&
+                off + width <= in.size(1) && out_off >= 0 && out_off + width <= out.size(1),
+            "activation_columns: the columns must lie inside in and out");
+  AKV_CHECK(kind >= 0 && kind <= akv::kActLast, "activation_columns: unknown activation");
+  c10::cuda::CUDAGuard guard(in.device());
+  check_launch(akv::launch_activation_columns(static_cast<const char*>(in.data_ptr()) + off * in.element_size(),
+                                              static_cast<char*>(out.data_ptr()) + out_off * out.element_size(), in.size(0),
+                                              (int)width, in.size(1), out.size(1), (int)kind, dtype_code(in, "in"),
+                                              stream_of(in)), "activation_columns");
+}
+
+void stream_sum(Tensor& hidden, const OptTensor& a, const OptTensor& b, const OptTensor& parts, const OptTensor& shared,
+                int64_t top, const OptTensor& copy) {
+  check_f32(hidden, "hidden");
+  AKV_CHECK(hidden.dim() == 2, "hidden must be [tokens, width]");
+  const int64_t n = hidden.numel();
+  akv::StreamSumParams p{};
+  p.hidden = hidden.data_ptr<float>();
+  p.num_tokens = hidden.size(0);
+  p.width = (int)hidden.size(1);
+  auto take = [&](const OptTensor& t, const char* name, const void** ptr, int* code) {
+    if (!t.has_value()) return;
+    check_cuda(*t, name);
+    AKV_CHECK(t->numel() == n && t->device() == hidden.device(), name, " must be [tokens, width] on the stream's device");
+    *ptr = t->data_ptr();
+    *code = dtype_code(*t, name);
+  };
+  take(a, "a", &p.a, &p.a_dtype);
+  take(b, "b", &p.b, &p.b_dtype);
+  if (parts.has_value()) {
+    AKV_CHECK(top >= 1, "stream_sum: top must be positive");
+    check_f32(*parts, "parts", n * top);
+    p.parts = parts->data_ptr<float>();
+    p.top = (int)top;
+    take(shared, "shared", &p.shared, &p.shared_dtype);
+  }
+  const void* copy_ptr = nullptr;
+  take(copy, "copy", &copy_ptr, &p.copy_dtype);
+  p.copy = const_cast<void*>(copy_ptr);
+  c10::cuda::CUDAGuard guard(hidden.device());
+  check_launch(akv::launch_stream_sum(p, stream_of(hidden)), "stream_sum");
+}
+
+void stream_concat(const Tensor& hidden, const Tensor& start, Tensor& out) {
+  check_f32(hidden, "hidden");
+  check_f32(start, "start", hidden.numel());
+  check_cuda(out, "out");
+  AKV_CHECK(hidden.dim() == 2 && out.dim() == 2 && out.size(0) == hidden.size(0) && out.size(1) == 2 * hidden.size(1),
+            "stream_concat: out must be [tokens, 2 * width]");
+  c10::cuda::CUDAGuard guard(hidden.device());
+  check_launch(akv::launch_stream_concat(hidden.data_ptr<float>(), start.data_ptr<float>(), out.data_ptr(), hidden.size(0),
+                                         (int)hidden.size(1), dtype_code(out, "out"), stream_of(hidden)), "stream_concat");
+}
+
+void stream_row_add(Tensor& hidden, const Tensor& row) {
+  check_f32(hidden, "hidden");
+  AKV_CHECK(hidden.dim() == 2, "hidden must be [tokens, width]");
+  check_f32(row, "row", hidden.size(1));
+  c10::cuda::CUDAGuard guard(hidden.device());
+  check_launch(akv::launch_stream_row_add(hidden.data_ptr<float>(), row.data_ptr<float>(), hidden.size(0),
+                                          (int)hidden.size(1), stream_of(hidden)), "stream_row_add");
+}
+
+void token_gate(const Tensor& z, const Tensor& ids, const OptTensor& sampled, const Tensor& table, int64_t col_off,
+                Tensor& out, const OptTensor& status) {
+  check_cuda(z, "z");
+  check_cuda(table, "table");
+  check_cuda(out, "out");
+  check_same(z, table, "z", "table");
+  check_same(z, out, "z", "out");
+  AKV_CHECK(z.dim() == 2 && table.dim() == 2 && out.sizes() == z.sizes() && col_off >= 0 &&
+                col_off + z.size(1) <= table.size(1), "token_gate: z and out [tokens, dim], the columns inside the table");
+  check_i32(ids, "ids");
+  AKV_CHECK(ids.numel() == z.size(0), "token_gate: an id per token");
+  akv::TokenGateParams p{};
+  p.z = z.data_ptr();
+  p.ids = ids.data_ptr<int>();
+  if (sampled.has_value()) {
+    check_i32(*sampled, "sampled");
+    p.sampled = sampled->data_ptr<int>();
+    p.num_sampled = sampled->numel();
+  }
+  p.table = table.data_ptr();
+  p.out = out.data_ptr();
+  p.num_tokens = z.size(0);
+  p.table_stride = table.size(1);
+  p.col_off = col_off;
+  p.vocab = table.size(0);
+  p.dim = (int)z.size(1);
+  p.dtype = dtype_code(z, "z");
+  p.status = status_ptr(status);
+  c10::cuda::CUDAGuard guard(z.device());
+  check_launch(akv::launch_token_gate(p, stream_of(z)), "token_gate");
+}
+
 void moe_route(const Tensor& logits, const OptTensor& correction, Tensor& chosen, Tensor& weights, int64_t groups,
                int64_t keep_groups, int64_t group_top, double scale, double weight_eps, int64_t score_kind,
-               bool normalize) {
+               bool normalize, const OptTensor& bias) {
   check_cuda(logits, "logits");
   AKV_CHECK(logits.scalar_type() == at::kFloat && logits.dim() == 2, "logits must be float32 [tokens, experts]");
   const int64_t n = logits.size(0), experts = logits.size(1);
@@ -1762,6 +2034,10 @@ void moe_route(const Tensor& logits, const OptTensor& correction, Tensor& chosen
   if (correction.has_value()) {
     check_f32(*correction, "correction", experts);
     p.correction = correction->data_ptr<float>();
+  }
+  if (bias.has_value()) {
+    check_f32(*bias, "bias", experts);
+    p.bias = bias->data_ptr<float>();
   }
   p.chosen = chosen.data_ptr<int>();
   p.weights = weights.data_ptr<float>();
@@ -1837,7 +2113,41 @@ void moe_gate_up(const Tensor& x, const Tensor& w, const Tensor& order, const Te
   AKV_CHECK(form >= 0 && form <= 3, "form: 0 by size, 1 float arithmetic, 2 mma.sync tiles, 3 few rows");
   p.force_plain = (int)form;
   c10::cuda::CUDAGuard guard(x.device());
-  check_launch(akv::launch_moe_gemm(p, true, stream_of(x)), "moe_gate_up");
+  check_launch(akv::launch_moe_gemm(p, akv::kMoeGated, stream_of(x)), "moe_gate_up");
+}
+
+// act[r] = activation(w[expert of sorted row r] x[token of that row]): experts without a gate.
+void moe_up(const Tensor& x, const Tensor& w, const Tensor& order, const Tensor& offsets, Tensor& act, int64_t top,
+            int64_t activation, int64_t form) {
+  check_cuda(x, "x");
+  check_cuda(w, "w");
+  check_cuda(act, "act");
+  check_same(x, w, "x", "w");
+  check_same(x, act, "x", "act");
+  AKV_CHECK(x.dim() == 2 && w.dim() == 3 && w.size(2) == x.size(1), "moe_up: x [tokens, hidden], w [experts, intermediate, hidden]");
+  const int64_t pairs = order.numel(), experts = w.size(0), inter = w.size(1);
+  check_i32(order, "order");
+  check_i32(offsets, "offsets", experts + 1);
+  AKV_CHECK(top >= 1 && pairs == x.size(0) * top && act.numel() == pairs * inter,
+            "moe_up: order holds tokens * top pairs, act [pairs, intermediate]");
+  AKV_CHECK(activation >= 0 && activation <= akv::kActLast, "moe_up: unknown activation");
+  AKV_CHECK(form >= 0 && form <= 3, "form: 0 by size, 1 float arithmetic, 2 mma.sync tiles, 3 few rows");
+  akv::MoeGemmParams p{};
+  p.a = x.data_ptr();
+  p.w = w.data_ptr();
+  p.order = order.data_ptr<int>();
+  p.offsets = offsets.data_ptr<int>();
+  p.out = act.data_ptr();
+  p.pairs = pairs;
+  p.experts = (int)experts;
+  p.k = (int)x.size(1);
+  p.n = (int)inter;
+  p.top = (int)top;
+  p.activation = (int)activation;
+  p.dtype = dtype_code(x, "x");
+  p.force_plain = (int)form;
+  c10::cuda::CUDAGuard guard(x.device());
+  check_launch(akv::launch_moe_gemm(p, akv::kMoeUp, stream_of(x)), "moe_up");
 }
 
 void moe_down(const Tensor& act, const Tensor& w, const Tensor& order, const Tensor& offsets, const Tensor& weights,
@@ -1868,7 +2178,7 @@ void moe_down(const Tensor& act, const Tensor& w, const Tensor& order, const Ten
   AKV_CHECK(form >= 0 && form <= 3, "form: 0 by size, 1 float arithmetic, 2 mma.sync tiles, 3 few rows");
   p.force_plain = (int)form;
   c10::cuda::CUDAGuard guard(act.device());
-  check_launch(akv::launch_moe_gemm(p, false, stream_of(act)), "moe_down");
+  check_launch(akv::launch_moe_gemm(p, akv::kMoeDown, stream_of(act)), "moe_down");
 }
 
 void moe_combine(const Tensor& parts, const OptTensor& shared, Tensor& out, int64_t top, const OptTensor& chosen,
@@ -1981,7 +2291,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("num_heads"), py::arg("num_kv_heads"), py::arg("v_dim"), py::arg("window"), py::arg("chunk"),
         py::arg("scale"), py::arg("softcap"), py::arg("slopes") = py::none(), py::arg("gate") = py::none(),
         py::arg("status") = py::none(), py::arg("kernel") = 0, py::arg("keep_first") = 0, py::arg("sigmoid_weights") = false,
-        py::arg("head_bias") = py::none(), py::arg("out_scale") = 1.0);
+        py::arg("head_bias") = py::none(), py::arg("out_scale") = 1.0, py::arg("sink") = py::none());
   m.def("head_prep", &head_prep, py::arg("x"), py::arg("slots"), py::arg("q_out"), py::arg("k_cache"),
         py::arg("v_cache"), py::arg("v_keep"), py::arg("v_other"), py::arg("blend_weight"), py::arg("gate_out"),
         py::arg("num_heads"), py::arg("num_kv_heads"), py::arg("head_dim"), py::arg("v_dim"), py::arg("unit_norm"),
@@ -2012,10 +2322,14 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("softcap", &softcap, py::arg("logits"), py::arg("cap"));
   m.def("delta_prep", &delta_prep, py::arg("x"), py::arg("conv"), py::arg("rate_log"), py::arg("step_bias"),
         py::arg("state"), py::arg("cu_q"), py::arg("state_slots"), py::arg("qkv"), py::arg("coef"), py::arg("num_heads"),
-        py::arg("num_kv_heads"), py::arg("head_dim"), py::arg("v_dim"), py::arg("taps"), py::arg("unit_eps"));
+        py::arg("num_kv_heads"), py::arg("head_dim"), py::arg("v_dim"), py::arg("taps"), py::arg("unit_eps"),
+        py::arg("steps") = py::none(), py::arg("step_off") = 0, py::arg("channel_decay") = false, py::arg("x_off") = 0,
+        py::arg("beta_off") = 0);
   m.def("delta_scan", &delta_scan, py::arg("qkv"), py::arg("coef"), py::arg("x"), py::arg("norm_weight"), py::arg("state"),
         py::arg("cu_q"), py::arg("state_slots"), py::arg("scratch"), py::arg("out"), py::arg("num_heads"),
-        py::arg("num_kv_heads"), py::arg("head_dim"), py::arg("v_dim"), py::arg("taps"), py::arg("norm_eps"));
+        py::arg("num_kv_heads"), py::arg("head_dim"), py::arg("v_dim"), py::arg("taps"), py::arg("norm_eps"),
+        py::arg("gates") = py::none(), py::arg("gate_off") = 0, py::arg("gate_kind") = 0, py::arg("channel_decay") = false,
+        py::arg("x_off") = 0, py::arg("out_off") = 0, py::arg("factor") = 1.0);
   m.def("delta_scan_supported", [](int64_t dim, int64_t v_dim) { return akv::delta_scan_supported((int)dim, (int)v_dim); });
   m.def("delta_memory_floats", [](int64_t heads, int64_t dim, int64_t v_dim) {
     return akv::delta_memory_floats((int)heads, (int)dim, (int)v_dim);
@@ -2057,15 +2371,32 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("out"), py::arg("num_heads"), py::arg("v_dim"), py::arg("state_dim"), py::arg("groups"), py::arg("taps"),
         py::arg("conv_off"), py::arg("step_off"));
   m.def("conv_tail", &conv_tail, py::arg("x"), py::arg("state"), py::arg("tail_off"), py::arg("cu_q"),
-        py::arg("state_slots"), py::arg("conv_off"), py::arg("channels"), py::arg("taps"));
+        py::arg("state_slots"), py::arg("conv_off"), py::arg("channels"), py::arg("taps"), py::arg("bias") = py::none());
+  m.def("conv_rotary_prep", &conv_rotary_prep, py::arg("x"), py::arg("x_off"), py::arg("bias"), py::arg("conv"),
+        py::arg("state"), py::arg("tail_off"), py::arg("cu_q"), py::arg("state_slots"), py::arg("positions"),
+        py::arg("slots"), py::arg("freq"), py::arg("q_out"), py::arg("k_cache"), py::arg("v_cache"), py::arg("num_heads"),
+        py::arg("num_kv_heads"), py::arg("head_dim"), py::arg("v_dim"), py::arg("taps"), py::arg("rotary_dims"),
+        py::arg("layout"), py::arg("factor"), py::arg("keep_tail"), py::arg("status") = py::none());
+  m.def("gate_columns", &gate_columns, py::arg("in"), py::arg("x"), py::arg("gate_off"), py::arg("out"),
+        py::arg("out_off"), py::arg("factor") = 1.0);
+  m.def("activation_columns", &activation_columns, py::arg("in"), py::arg("off"), py::arg("width"), py::arg("kind"),
+        py::arg("out"), py::arg("out_off"));
+  m.def("stream_sum", &stream_sum, py::arg("hidden"), py::arg("a"), py::arg("b"), py::arg("parts"), py::arg("shared"),
+        py::arg("top"), py::arg("copy"));
+  m.def("stream_concat", &stream_concat, py::arg("hidden"), py::arg("start"), py::arg("out"));
+  m.def("stream_row_add", &stream_row_add, py::arg("hidden"), py::arg("row"));
+  m.def("token_gate", &token_gate, py::arg("z"), py::arg("ids"), py::arg("sampled"), py::arg("table"), py::arg("col_off"),
+        py::arg("out"), py::arg("status") = py::none());
   m.def("scaled_sum", &scaled_sum, py::arg("a"), py::arg("b"), py::arg("out"), py::arg("sa"), py::arg("sb"));
   m.def("moe_route", &moe_route, py::arg("logits"), py::arg("correction"), py::arg("chosen"), py::arg("weights"),
         py::arg("groups"), py::arg("keep_groups"), py::arg("group_top"), py::arg("scale"), py::arg("weight_eps"),
-        py::arg("score_kind") = 0, py::arg("normalize") = true);
+        py::arg("score_kind") = 0, py::arg("normalize") = true, py::arg("bias") = py::none());
   m.def("moe_router", &moe_router, py::arg("x"), py::arg("w"), py::arg("logits"));
   m.def("moe_sort", &moe_sort, py::arg("chosen"), py::arg("order"), py::arg("offsets"));
   m.def("moe_gate_up", &moe_gate_up, py::arg("x"), py::arg("w"), py::arg("order"), py::arg("offsets"), py::arg("act"),
         py::arg("top"), py::arg("limit"), py::arg("slope"), py::arg("form") = 0, py::arg("up_offset") = 1.0);
+  m.def("moe_up", &moe_up, py::arg("x"), py::arg("w"), py::arg("order"), py::arg("offsets"), py::arg("act"),
+        py::arg("top"), py::arg("activation"), py::arg("form") = 0);
   m.def("moe_down", &moe_down, py::arg("act"), py::arg("w"), py::arg("order"), py::arg("offsets"), py::arg("weights"),
         py::arg("out"), py::arg("form") = 0);
   m.def("moe_combine", &moe_combine, py::arg("parts"), py::arg("shared"), py::arg("out"), py::arg("top"),

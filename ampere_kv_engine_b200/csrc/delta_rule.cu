@@ -3,14 +3,16 @@
 //   delta_prep:  one product holds [q | k | v | gate | beta | step] of every token.  q, k and v pass a short causal
 //                convolution over the sequence's own earlier tokens (the inputs before the step's first token come
 //                from the request's state slot) and SiLU; q and k heads become unit vectors (q also times
-//                dim^-1/2); beta = sigmoid(.), decay = exp(-exp(rate_log) * softplus(step + step_bias)).
-//                Everything it writes is float32.  One warp per (token, head).
+//                dim^-1/2); beta = sigmoid(.), decay = exp(-exp(rate_log) * softplus(step + step_bias)), one per head
+//                or, with channel_decay, one per head and key channel (it then multiplies the rows of S).  Gate and
+//                step may come from a product of their own.  Everything it writes is float32.  One warp per
+//                (token, head).
 //   delta_scan:  blocks per (sequence, head, slice of the value columns) walk the step's tokens of that sequence in
 //                order:  S *= decay;  u = beta (v - S^T k);  S += k u^T;  o = S^T q.
 //                A thread group of up to 8 lanes owns one value column of S (in registers for the whole step); the
 //                two products are a few multiply-adds per lane and a shuffle reduction over the group; tokens are
 //                staged through shared memory in chunks, so a token costs no block barrier.  A second kernel applies
-//                the output norm o / sqrt(mean(o^2) + eps) * w * silu(gate) to all tokens in parallel and, in further
+//                the output norm o / sqrt(mean(o^2) + eps) * w * silu(gate) (or sigmoid(gate)) to all tokens in parallel and, in further
 //                blocks, moves each sequence's last taps - 1 convolution inputs into the state.
 //
 // The walk is token by token whatever the step holds, so the state after a token does not depend on how the
@@ -37,6 +39,10 @@ __device__ __forceinline__ int sequence_of(const int32_t* cu_q, int num_seqs, in
 
 constexpr int kMaxPerLane = kDeltaMaxDim / 32;
 
+__device__ __forceinline__ float load_any(const void* p, int64_t i, int dtype) {
+  return dtype == kBFloat16 ? __bfloat162float(((const __nv_bfloat16*)p)[i]) : ((const float*)p)[i];
+}
+
 }  // namespace
 
 template <typename T>
@@ -45,27 +51,40 @@ __global__ void delta_prep_kernel(DeltaParams p) {
   pdl_wait();
   const int lane = threadIdx.x & 31;
   const int G = p.num_kv_heads, H = p.num_heads, D = p.head_dim, V = p.v_dim;
-  const int units = 2 * G + H + 1;
+  const int units = 2 * G + H + 1 + (p.channel_decay ? H : 0);
   const int64_t item = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (item >= p.num_tokens * units) return;
   const int64_t token = item / units;
   const int unit = (int)(item - token * units);
   const int channels = 2 * G * D + H * V;
-  const int64_t width = (int64_t)channels + (int64_t)H * V + 2 * H;
-  const T* x = (const T*)p.x;
+  const int64_t width = p.x_stride;
+  const T* x = (const T*)p.x + p.x_off;
   const int s = sequence_of(p.cu_q, p.num_seqs, token);
   const int slot = p.state_slots[s];
-  float* coef = p.coef + token * 2 * H;
-  if (unit == units - 1) {
+  const bool held = slot >= 0 && slot < p.num_slots;
+  float* coef = p.coef + token * p.coef_stride;
+  if (unit == 2 * G + H) {
+    const int64_t step0 = token * p.step_stride + p.step_off;
     for (int h = lane; h < H; h += 32) {
-      float beta = 0.f, decay = 0.f;
-      if (slot >= 0 && slot < p.num_slots) {
-        const T* tail = x + token * width + channels + (int64_t)H * V;
-        beta = 1.f / (1.f + expf(-to_float<T>(tail[h])));
-        decay = expf(-expf(p.rate_log[h]) * softplus(to_float<T>(tail[H + h]) + p.step_bias[h]));
-      }
+      float beta = 0.f;
+      if (held) beta = 1.f / (1.f + expf(-to_float<T>(((const T*)p.x)[token * width + p.beta_off + h])));
       coef[h] = beta;
-      coef[H + h] = decay;
+      if (!p.channel_decay) {
+        float decay = 0.f;
+        if (held) decay = expf(-expf(p.rate_log[h]) * softplus(load_any(p.steps, step0 + h, p.step_dtype) + p.step_bias[h]));
+        coef[H + h] = decay;
+      }
+    }
+    return;
+  }
+  if (unit > 2 * G + H) {
+    const int h = unit - (2 * G + H + 1);
+    const float rate = expf(p.rate_log[h]);
+    const int64_t step0 = token * p.step_stride + p.step_off + (int64_t)h * D;
+    for (int d = lane; d < D; d += 32) {
+      float decay = 0.f;
+      if (held) decay = expf(-rate * softplus(load_any(p.steps, step0 + d, p.step_dtype) + p.step_bias[h * D + d]));
+      coef[H + h * D + d] = decay;
     }
     return;
   }
@@ -74,7 +93,7 @@ __global__ void delta_prep_kernel(DeltaParams p) {
   const int n = unit_vector ? D : V;
   const int first = unit_vector ? unit * D : 2 * G * D + (unit - 2 * G) * V;
   float* out = p.qkv + token * channels + first;
-  if (slot < 0 || slot >= p.num_slots) {
+  if (!held) {
     for (int d = lane; d < n; d += 32) out[d] = 0.f;
     return;
   }
@@ -119,7 +138,7 @@ int launch_delta_prep(const DeltaParams& p, cudaStream_t stream) {
   if (p.num_tokens == 0) return 0;
   if (p.head_dim > kDeltaMaxDim || p.v_dim > kDeltaMaxDim || p.taps < 1 || p.taps > kDeltaMaxTaps)
     return (int)cudaErrorInvalidValue;
-  const int units = 2 * p.num_kv_heads + p.num_heads + 1;
+  const int units = 2 * p.num_kv_heads + p.num_heads + 1 + (p.channel_decay ? p.num_heads : 0);
   const int warps = 4;
   const int64_t blocks = (p.num_tokens * units + warps - 1) / warps;
   if (blocks > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
@@ -144,14 +163,22 @@ struct ScanShape {
   int ept, lanes, cols, threads, chunk;   // elements per lane, lanes per column, columns and threads per block, tokens per chunk
 };
 
-// a thread stages up to kScanRounds entries of each of up to kScanChunk tokens (registers it holds of the chunk
-// under way)
-constexpr int kScanRounds = 3, kScanChunk = 16;
+// a thread stages up to kScanRounds entries (kWideRounds where a lane holds 32 elements and the decays are per channel)
+// of each of up to kScanChunk tokens (registers it holds of the chunk under way)
+constexpr int kScanRounds = 3, kWideRounds = 4, kScanChunk = 16;
+__host__ __device__ constexpr int scan_rounds(int ept, bool channel) {
+  return channel && ept >= 32 ? kWideRounds : kScanRounds;
+}
 
-// floats of one staged token in shared memory: q and k (each lane's elements padded by four floats), the block's v
-// columns, beta and decay; a multiple of four, so that every token's q and k can be read as float4
-__host__ __device__ inline int scan_token_floats(int lanes, int ept, int cols) {
-  return (2 * lanes * (ept + 4) + cols + 2 + 3) / 4 * 4;
+// floats of one staged token in shared memory: q and k (and the decays, if each key channel has its own; each lane's
+// elements padded by four floats), the block's v columns, beta and decay; a multiple of four, so that every token's q
+// and k can be read as float4
+__host__ __device__ inline int scan_token_floats(int lanes, int ept, int cols, bool channel) {
+  return ((channel ? 3 : 2) * lanes * (ept + 4) + cols + 2 + 3) / 4 * 4;
+}
+// entries of a token that a block stages
+__host__ __device__ inline int scan_entries(int dim, int cols, bool channel) {
+  return channel ? 3 * dim + cols + 1 : 2 * dim + cols + 2;
 }
 
 __host__ __device__ inline int pow2_at_least(int n) {
@@ -163,7 +190,7 @@ __host__ __device__ inline int pow2_at_least(int n) {
 // the smallest EPT of 4, 8, 16, 32 with which 8 lanes cover the dim; 256 threads a block.  (Narrower slices of the
 // value columns, so that a single sequence's blocks cover all SMs, were measured and not kept: a block's time per
 // token is the chain of one token's latencies whatever its width, 0.31 us at 16 and at 32 columns.)
-inline ScanShape scan_shape(int dim, int v_dim) {
+inline ScanShape scan_shape(int dim, int v_dim, bool channel = false) {
   ScanShape s{0, 0, 0, 0, 0};
   for (int e : {4, 8, 16, 32}) {
     const int lanes = pow2_at_least((dim + e - 1) / e);
@@ -178,12 +205,13 @@ inline ScanShape scan_shape(int dim, int v_dim) {
   if (s.cols > v_dim) s.cols = v_dim;
   s.threads = (s.cols * s.lanes + 31) / 32 * 32;
   if (s.threads < 128) s.threads = 128;      // the fetch of a chunk is spread over the block (threads without a column idle)
-  // a token's entries must fit in kScanRounds rounds of the block
-  while (s.threads * kScanRounds < 2 * dim + s.cols + 2) s.threads += 32;
-  // the chunk of a prompt: 16 tokens, 8 where a lane holds 32 elements (two buffers within 48 KB)
-  const int per_token = scan_token_floats(s.lanes, s.ept, s.cols);
+  // a token's entries must fit in the block's rounds
+  while (s.threads * scan_rounds(s.ept, channel) < scan_entries(dim, s.cols, channel)) s.threads += 32;
+  // the chunk of a prompt: 16 tokens, 8 where a lane holds 32 elements (two buffers within 48 KB, or 72 KB with the
+  // decays of every channel)
+  const int per_token = scan_token_floats(s.lanes, s.ept, s.cols, channel);
   s.chunk = kScanChunk;
-  while (s.chunk > 1 && 2 * s.chunk * per_token * 4 > 48 * 1024) s.chunk /= 2;
+  while (s.chunk > 1 && 2 * s.chunk * per_token * 4 > (channel ? 72 : 48) * 1024) s.chunk /= 2;
   if (s.ept >= 32 && s.chunk > 8) s.chunk = 8;
   return s;
 }
@@ -199,8 +227,9 @@ int64_t delta_memory_floats(int num_heads, int dim, int v_dim) {
   return (int64_t)num_heads * v_dim * s.lanes * s.ept;
 }
 
-template <int EPT, int LANES, int CHUNK>
+template <int EPT, int LANES, int CHUNK, bool CHANNEL>
 __global__ void __launch_bounds__(256) delta_scan_kernel(DeltaParams p, int cols) {
+  constexpr int kRounds = scan_rounds(EPT, CHANNEL);
   constexpr int chunk = CHUNK;
   extern __shared__ __align__(16) float smem[];
   constexpr int kPitch = EPT + 4;      // a lane's elements of q or k, padded: the lanes of a group read different banks
@@ -235,24 +264,27 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(DeltaParams p, int cols
   }
 
   constexpr int vec = lanes * kPitch;                                 // floats of one token's q (or k) in shared memory
-  const int per_token = scan_token_floats(lanes, EPT, cols);      // q, k, v of the block's columns, beta, decay
+  // q, k (the channels' decays), v of the block's columns, beta (, decay)
+  const int per_token = scan_token_floats(lanes, EPT, cols, CHANNEL);
+  constexpr int v_at = (CHANNEL ? 3 : 2) * vec;
   const int per_buffer = chunk * per_token;
-  // What a thread stages of every token: entry i = threadIdx.x + round * blockDim.x of [q | k | v | beta | decay].
+  // What a thread stages of every token: entry i = threadIdx.x + round * blockDim.x of [q | k | v | beta | decay], the
+  // last of which is one number or the key width of them.
   // Where it comes from (a column of the token's qkv or coef row) and where it goes in the token's shared-memory row
   // are worked out once; a chunk is then one load per (round, token).
-  const int fetch_per_token = 2 * D + mine_cols + 2;
-  const float* src[kScanRounds];
-  int src_stride[kScanRounds], dst[kScanRounds];
+  const int fetch_per_token = scan_entries(D, mine_cols, CHANNEL);
+  const float* src[kRounds];
+  int src_stride[kRounds], dst[kRounds];
 #pragma unroll
-  for (int r = 0; r < kScanRounds; ++r) {
+  for (int r = 0; r < kRounds; ++r) {
     const int i = threadIdx.x + r * blockDim.x;
     src[r] = nullptr;
     src_stride[r] = 0;
     dst[r] = 0;
     if (i < fetch_per_token) {
       const float* qkv = p.qkv + first * channels;
-      const float* coef = p.coef + first * 2 * H;
-      src_stride[r] = i < 2 * D + mine_cols ? channels : 2 * H;
+      const float* coef = p.coef + first * p.coef_stride;
+      src_stride[r] = i < 2 * D + mine_cols ? channels : (int)p.coef_stride;
       if (i < D) {
         src[r] = qkv + g * D + i;
         dst[r] = i / EPT * kPitch + i % EPT;
@@ -261,17 +293,24 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(DeltaParams p, int cols
         dst[r] = vec + (i - D) / EPT * kPitch + (i - D) % EPT;
       } else if (i < 2 * D + mine_cols) {
         src[r] = qkv + 2 * G * D + h * V + col0 + (i - 2 * D);
-        dst[r] = 2 * vec + (i - 2 * D);
+        dst[r] = v_at + (i - 2 * D);
+      } else if (i == 2 * D + mine_cols) {
+        src[r] = coef + h;
+        dst[r] = v_at + cols;
+      } else if (CHANNEL) {
+        const int d = i - 2 * D - mine_cols - 1;
+        src[r] = coef + H + h * D + d;
+        dst[r] = 2 * vec + d / EPT * kPitch + d % EPT;
       } else {
-        src[r] = coef + (i == 2 * D + mine_cols ? h : H + h);
-        dst[r] = 2 * vec + cols + (i - 2 * D - mine_cols);
+        src[r] = coef + H + h;
+        dst[r] = v_at + cols + 1;
       }
     }
   }
-  float regs[kScanRounds][CHUNK];
+  float regs[kRounds][CHUNK];
   auto fetch = [&](int t0, int count) {
 #pragma unroll
-    for (int r = 0; r < kScanRounds; ++r) {
+    for (int r = 0; r < kRounds; ++r) {
 #pragma unroll
       for (int t = 0; t < CHUNK; ++t) {
         regs[r][t] = 0.f;
@@ -281,7 +320,7 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(DeltaParams p, int cols
   };
   auto stash = [&](float* buffer, int count) {
 #pragma unroll
-    for (int r = 0; r < kScanRounds; ++r) {
+    for (int r = 0; r < kRounds; ++r) {
 #pragma unroll
       for (int t = 0; t < CHUNK; ++t)
         if (src[r] != nullptr && t < count) buffer[t * per_token + dst[r]] = regs[r][t];
@@ -305,17 +344,30 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(DeltaParams p, int cols
     for (int t = 0; t < count; ++t, row += per_token, o_row += H * V) {
       const float* q = row + l * kPitch;
       const float* k = row + vec + l * kPitch;
-      const float v = owner ? row[2 * vec + col] : 0.f;
-      const float beta = row[2 * vec + cols], decay = row[2 * vec + cols + 1];
+      const float v = owner ? row[v_at + col] : 0.f;
+      const float beta = row[v_at + cols];
       float kr[EPT];
       float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
+      float decay = 1.f;
+      if constexpr (CHANNEL) {
+        // every row of S by its own decay first; what follows is then the form with one decay, at one
+        const float* g = row + 2 * vec + l * kPitch;
+#pragma unroll
+        for (int e = 0; e < EPT; e += 4) {
+          const float4 gg = *reinterpret_cast<const float4*>(g + e);
+          S[e] *= gg.x; S[e + 1] *= gg.y; S[e + 2] *= gg.z; S[e + 3] *= gg.w;
+        }
+      } else {
+        decay = row[v_at + cols + 1];
+      }
 #pragma unroll
       for (int e = 0; e < EPT; e += 4) {
         const float4 kk = *reinterpret_cast<const float4*>(k + e);
         kr[e] = kk.x; kr[e + 1] = kk.y; kr[e + 2] = kk.z; kr[e + 3] = kk.w;
         a0 = fmaf(S[e], kk.x, a0); a1 = fmaf(S[e + 1], kk.y, a1); a2 = fmaf(S[e + 2], kk.z, a2); a3 = fmaf(S[e + 3], kk.w, a3);
       }
-      float kv = ((a0 + a1) + (a2 + a3)) * decay;           // (decay S)^T k
+      float kv = (a0 + a1) + (a2 + a3);                     // (decay S)^T k
+      if constexpr (!CHANNEL) kv *= decay;
 #pragma unroll
       for (int o = lanes >> 1; o > 0; o >>= 1) kv += __shfl_xor_sync(0xffffffffu, kv, o);
       const float u = beta * (v - kv);
@@ -323,8 +375,13 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(DeltaParams p, int cols
 #pragma unroll
       for (int e = 0; e < EPT; e += 4) {
         const float4 qq = *reinterpret_cast<const float4*>(q + e);
-        S[e] = fmaf(kr[e], u, S[e] * decay); S[e + 1] = fmaf(kr[e + 1], u, S[e + 1] * decay);
-        S[e + 2] = fmaf(kr[e + 2], u, S[e + 2] * decay); S[e + 3] = fmaf(kr[e + 3], u, S[e + 3] * decay);
+        if constexpr (CHANNEL) {
+          S[e] = fmaf(kr[e], u, S[e]); S[e + 1] = fmaf(kr[e + 1], u, S[e + 1]);
+          S[e + 2] = fmaf(kr[e + 2], u, S[e + 2]); S[e + 3] = fmaf(kr[e + 3], u, S[e + 3]);
+        } else {
+          S[e] = fmaf(kr[e], u, S[e] * decay); S[e + 1] = fmaf(kr[e + 1], u, S[e + 1] * decay);
+          S[e + 2] = fmaf(kr[e + 2], u, S[e + 2] * decay); S[e + 3] = fmaf(kr[e + 3], u, S[e + 3] * decay);
+        }
         a0 = fmaf(S[e], qq.x, a0); a1 = fmaf(S[e + 1], qq.y, a1); a2 = fmaf(S[e + 2], qq.z, a2); a3 = fmaf(S[e + 3], qq.w, a3);
       }
       float o = (a0 + a1) + (a2 + a3);
@@ -343,7 +400,7 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(DeltaParams p, int cols
 }
 
 // What follows the scan, in one launch.  Blocks [0, norm_blocks): the output norm and gate, a warp per (token, head):
-// o / sqrt(mean(o^2) + eps) * w * silu(gate).  The blocks after them: the convolutions' memory, a thread per
+// o / sqrt(mean(o^2) + eps) * w * silu(gate) or sigmoid(gate), times a factor.  The blocks after them: the convolutions' memory, a thread per
 // (sequence, channel): the last taps - 1 inputs of [what was there before | this step's rows]; a thread reads all it
 // needs before it writes.
 template <typename T>
@@ -352,8 +409,8 @@ __global__ void __launch_bounds__(128) delta_finish_kernel(DeltaParams p, int no
   pdl_wait();
   const int H = p.num_heads, V = p.v_dim;
   const int channels = 2 * p.num_kv_heads * p.head_dim + H * V;
-  const int64_t width = (int64_t)channels + (int64_t)H * V + 2 * H;
-  const T* x = (const T*)p.x;
+  const int64_t width = p.x_stride;
+  const T* x = (const T*)p.x + p.x_off;
   if ((int)blockIdx.x < norm_blocks) {
     const int lane = threadIdx.x & 31;
     const int64_t item = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -364,11 +421,12 @@ __global__ void __launch_bounds__(128) delta_finish_kernel(DeltaParams p, int no
     float ss = 0.f;
     for (int j = lane; j < V; j += 32) ss += raw[j] * raw[j];
     const float inv = rsqrtf(warp_sum(ss) / (float)V + p.norm_eps);
-    const T* gate = x + token * width + channels + (int64_t)h * V;
-    T* dst = (T*)p.out + token * H * V + (int64_t)h * V;
+    const int64_t gate0 = token * p.gate_stride + p.gate_off + (int64_t)h * V;
+    T* dst = (T*)p.out + token * p.out_stride + p.out_off + (int64_t)h * V;
     for (int j = lane; j < V; j += 32) {
-      const float z = to_float<T>(gate[j]);
-      dst[j] = from_float<T>(raw[j] * inv * p.norm_weight[j] * (z / (1.f + expf(-z))));
+      const float z = load_any(p.gates, gate0 + j, p.gate_dtype);
+      const float g = (p.gate_kind == 1 ? 1.f : z) / (1.f + expf(-z));
+      dst[j] = from_float<T>(raw[j] * inv * p.norm_weight[j] * g * p.factor);
     }
     return;
   }
@@ -395,12 +453,12 @@ __global__ void __launch_bounds__(128) delta_finish_kernel(DeltaParams p, int no
     if (i < keep) before[(int64_t)i * channels + c] = kept[i];
 }
 
-template <int EPT, int LANES, int CHUNK>
+template <int EPT, int LANES, int CHUNK, bool CHANNEL>
 static int launch_scan_chunk(const DeltaParams& p, const ScanShape& shape, cudaStream_t stream) {
   const int threads = shape.threads;
-  const int per_token = scan_token_floats(shape.lanes, EPT, shape.cols);
+  const int per_token = scan_token_floats(shape.lanes, EPT, shape.cols, CHANNEL);
   const size_t smem = 2 * (size_t)CHUNK * per_token * sizeof(float);
-  auto kernel = delta_scan_kernel<EPT, LANES, CHUNK>;
+  auto kernel = delta_scan_kernel<EPT, LANES, CHUNK, CHANNEL>;
   if (smem > 48 * 1024) {
     cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (err != cudaSuccess) return (int)err;
@@ -412,20 +470,25 @@ static int launch_scan_chunk(const DeltaParams& p, const ScanShape& shape, cudaS
 
 // Steps of about a token per sequence (decoding) stage two tokens at a time: fewer registers and less shared memory
 // per block, so more blocks share an SM while the state streams through; prompts stage the largest chunk that fits.
+template <int EPT, int LANES, bool CHANNEL>
+static int launch_scan_form(const DeltaParams& p, const ScanShape& shape, cudaStream_t stream) {
+  constexpr int kLong = EPT >= 32 ? 8 : 16;
+  if (p.num_tokens <= 2 * (int64_t)p.num_seqs) return launch_scan_chunk<EPT, LANES, 2, CHANNEL>(p, shape, stream);
+  if (shape.chunk < kLong) return (int)cudaErrorInvalidValue;
+  return launch_scan_chunk<EPT, LANES, kLong, CHANNEL>(p, shape, stream);
+}
 template <int EPT, int LANES>
 static int launch_scan(const DeltaParams& p, const ScanShape& shape, cudaStream_t stream) {
-  constexpr int kLong = EPT >= 32 ? 8 : 16;
-  if (p.num_tokens <= 2 * (int64_t)p.num_seqs) return launch_scan_chunk<EPT, LANES, 2>(p, shape, stream);
-  if (shape.chunk < kLong) return (int)cudaErrorInvalidValue;
-  return launch_scan_chunk<EPT, LANES, kLong>(p, shape, stream);
+  return p.channel_decay ? launch_scan_form<EPT, LANES, true>(p, shape, stream)
+                         : launch_scan_form<EPT, LANES, false>(p, shape, stream);
 }
 
 int launch_delta_scan(const DeltaParams& p, cudaStream_t stream) {
   if (p.num_tokens == 0 || p.num_seqs == 0) return 0;
-  const ScanShape shape = scan_shape(p.head_dim, p.v_dim);
+  const ScanShape shape = scan_shape(p.head_dim, p.v_dim, p.channel_decay != 0);
   if (shape.ept == 0 || p.head_dim > kDeltaMaxDim || p.v_dim > kDeltaMaxDim || p.num_heads > 65535 ||
       p.memory != delta_memory_floats(p.num_heads, p.head_dim, p.v_dim) || shape.threads > 256 ||
-      shape.threads * kScanRounds < 2 * p.head_dim + shape.cols + 2 ||
+      shape.threads * scan_rounds(shape.ept, p.channel_decay != 0) < scan_entries(p.head_dim, shape.cols, p.channel_decay != 0) ||
       reinterpret_cast<uintptr_t>(p.state) % 16 != 0 || p.state_stride % 4 != 0)      // S moves as float4
     return (int)cudaErrorInvalidValue;
   int err;

@@ -641,12 +641,13 @@ EncodeTiledFn encode_fn() {
 }
 
 // Map over a row-major bfloat16 matrix [rows, cols]: boxes of 64 columns by `box_rows` rows, 128-byte swizzle,
-// zeros outside the matrix.
-bool matrix_map(const void* base, int64_t rows, int64_t cols, int box_rows, CUtensorMap* out) {
+// zeros outside the matrix.  row_stride: elements between two rows (0: cols).
+bool matrix_map(const void* base, int64_t rows, int64_t cols, int box_rows, CUtensorMap* out, int64_t row_stride = 0) {
+  if (row_stride == 0) row_stride = cols;
   static std::mutex mutex;
-  static std::map<std::tuple<const void*, int64_t, int64_t, int>, CUtensorMap> cache;
+  static std::map<std::tuple<const void*, int64_t, int64_t, int, int64_t>, CUtensorMap> cache;
   std::lock_guard<std::mutex> guard(mutex);
-  const auto key = std::make_tuple(base, rows, cols, box_rows);
+  const auto key = std::make_tuple(base, rows, cols, box_rows, row_stride);
   auto it = cache.find(key);
   if (it != cache.end()) {
     *out = it->second;
@@ -656,7 +657,7 @@ bool matrix_map(const void* base, int64_t rows, int64_t cols, int box_rows, CUte
   if (fn == nullptr) return false;
   CUtensorMap map;
   const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-  const cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
+  const cuuint64_t strides[1] = {(cuuint64_t)row_stride * 2};
   const cuuint32_t box[2] = {(cuuint32_t)kTileK, (cuuint32_t)box_rows};
   const cuuint32_t elem[2] = {1, 1};
   const CUresult res = fn(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box,
@@ -800,8 +801,8 @@ int launch_small_m_gemm(const void* x, const void* w, void* out, int out_dtype, 
   CUtensorMap w_map, x_map;
   if (!matrix_map(w, features, k, kTileM, &w_map)) return (int)cudaErrorInvalidValue;
   if (f.normed_x) x_map = w_map;      // unused
-  else if (!matrix_map(x, tokens, k, bn, &x_map)) return (int)cudaErrorInvalidValue;
-  if (f.activation >= 0 && (f.epilogue != kEpiloguePlain || out == nullptr || out_dtype != kBFloat16 || f.activation > 2))
+  else if (!matrix_map(x, tokens, k, bn, &x_map, f.x_stride)) return (int)cudaErrorInvalidValue;
+  if (f.activation >= 0 && (f.epilogue != kEpiloguePlain || out == nullptr || out_dtype != kBFloat16 || f.activation > kActLast))
     return (int)cudaErrorInvalidValue;
   GemmParams p{parts, out, (int)tokens, (int)features, (int)k, kb_total, splits, status, f.qkv, f.residual, f.normed,
                f.activation};

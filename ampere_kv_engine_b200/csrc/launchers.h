@@ -127,6 +127,7 @@ struct GemmFusion {
   // kEpiloguePlain with a bfloat16 out only: an Activation applied to the product (rounded to bfloat16 first, as the
   // stored product would be) before it is stored; -1: none
   int activation = -1;
+  int64_t x_stride = 0;      // elements between two rows of x (0: k)
 };
 int launch_small_m_gemm(const void* x, const void* w, void* out, int out_dtype, float* parts, int64_t tokens,
                         int64_t features, int64_t k, int splits, const GemmFusion* fusion, int* status,
@@ -237,6 +238,8 @@ struct ScoredAttentionParams {
   int sigmoid_weights;         // 1: a visible key weighs sigmoid(score + head_bias[h]); the weights are not normalised
   const float* head_bias;      // [NH] or null (read with sigmoid_weights)
   float out_scale;             // every output is multiplied by it (1: nothing)
+  const float* sink;           // [NH] or null: the softmax's denominator also counts exp(sink[h]), which has no key,
+                               // no value and no scale (not with sigmoid_weights)
 };
 int launch_scored_attention(const ScoredAttentionParams& p, cudaStream_t stream);
 // The tcgen05 prompt kernel's scored form (attention_tcgen05.cu): bfloat16 prompt tiles with keys and values of 128
@@ -341,8 +344,10 @@ struct BranchNormParams {
 constexpr int kBranchNormMaxTop = 32;
 int launch_branch_rmsnorm(const BranchNormParams& p, cudaStream_t stream);
 
-// The gated delta rule (delta_rule.cu).  x [N, q | k | v | gate | beta | step] with num_kv_heads heads of head_dim
-// for q and k, num_heads heads of v_dim for v and gate, one column per head for beta and step.  state
+// The gated delta rule (delta_rule.cu).  x [N, x_stride] holds q | k | v from column x_off (num_kv_heads heads of head_dim
+// for q and k, num_heads heads of v_dim for v) and one column per head for beta; the gate (num_heads * v_dim columns) and
+// the step (a column per head, or with channel_decay one per head and key channel) stand in x or in a tensor of their
+// own (low-rank projections).  state
 // [num_slots, state_stride] float32: per slot heads * v_dim * head_dim floats of S ([head][value column][dim]) at
 // offset 0 (in the scan kernel's own order, delta_memory_floats() of them) and (taps - 1) * channels convolution
 // inputs at offset `memory`.
@@ -358,13 +363,23 @@ struct DeltaParams {
   const int32_t* cu_q;         // [num_seqs + 1]
   const int32_t* state_slots;  // [num_seqs]; negative: the sequence is padding
   float* qkv;                  // [N, channels]: unit q, unit k, v
-  float* coef;                 // [N, 2 * num_heads]: beta, decay
+  float* coef;                 // [N, coef_stride]: beta per head, then decay per head (channel_decay: per head and
+                               // key channel)
   float* scratch;              // [N, num_heads * v_dim]: o before its norm
-  void* out;                   // [N, num_heads * v_dim]
+  void* out;                   // [N, out_stride], num_heads * v_dim columns from out_off
   int64_t num_tokens, state_stride, memory;
   int num_seqs, num_slots, num_heads, num_kv_heads, head_dim, v_dim, taps;
   float unit_eps, norm_eps;
   int dtype;
+  int64_t x_stride, coef_stride, out_stride;
+  int x_off, beta_off, out_off;
+  const void* gates;           // [N, gate_stride] of gate_dtype, from column gate_off
+  const void* steps;           // [N, step_stride] of step_dtype, from column step_off
+  int64_t gate_stride, step_stride;
+  int gate_off, gate_dtype, step_off, step_dtype;
+  int gate_kind;               // 0: SiLU, 1: sigmoid
+  int channel_decay;           // 1: a decay per head and key channel
+  float factor;                // on the normed, gated output
 };
 int launch_delta_prep(const DeltaParams& p, cudaStream_t stream);
 int launch_delta_scan(const DeltaParams& p, cudaStream_t stream);
@@ -383,6 +398,7 @@ struct MoeRouteParams {
   float scale, weight_eps;
   int score_kind;              // 0: sigmoid of each logit; 1: softmax over all experts
   int normalize;               // 1: the chosen scores are divided by their sum (plus weight_eps)
+  const float* bias;           // [experts] or null: added to the logits before the scores are formed
 };
 int launch_moe_route(const MoeRouteParams& p, cudaStream_t stream);
 // logits[t, e] = x[t, :] . w[e, :] in float, a warp per (token, expert): for steps of a few tokens.
@@ -391,32 +407,39 @@ int launch_moe_router(const void* x, const void* w, float* logits, int64_t token
 // order [pairs]: the (token, choice) pairs (token * top + choice) sorted by expert; offsets [experts + 1].
 int launch_moe_sort(const int32_t* chosen, int32_t* order, int32_t* offsets, int64_t pairs, int experts,
                     cudaStream_t stream);
+// The grouped products: kMoeDown, the second product of an expert, times the pair's weight; kMoeGated, the first of a
+// gated expert; kMoeUp, the first of one without a gate.
+enum MoeForm : int { kMoeDown = 0, kMoeGated = 1, kMoeUp = 2 };
 struct MoeGemmParams {
-  const void* a;               // gated: x [tokens, k]; else the activations [pairs, k] in sorted order
+  const void* a;               // gated, up: x [tokens, k]; else the activations [pairs, k] in sorted order
   const void* w;               // gated: [experts, 2 n, k] (gate rows, then up rows); else [experts, n, k]
   const int32_t* order;        // [pairs]
   const int32_t* offsets;      // [experts + 1]
-  const float* weights;        // [pairs] by pair (not gated)
-  void* out;                   // gated: [pairs, n] in sorted order, type of a; else float32 [pairs, n] by pair
+  const float* weights;        // [pairs] by pair (down)
+  void* out;                   // gated, up: [pairs, n] in sorted order, type of a; else float32 [pairs, n] by pair
   int64_t pairs;
   int experts, k, n, top;
   float limit, slope;
   float up_offset;             // the gated product's activation is g sigmoid(slope g) (u + up_offset)
   int dtype;
   int force_plain;             // 0: the form is chosen by size; 1: float arithmetic; 2: mma.sync tiles; 3: few rows
+  int activation;              // up: an Activation
 };
 // steps with at most this many (token, choice) pairs run the few-rows form of the gated product (measured at 8
 // tokens, 64 experts of 1,024 x 4,096: 103 against 111 us; the down product is faster in tiles: 59 against 89 us)
 constexpr int kMoeFewRowPairs = 128;
-int launch_moe_gemm(const MoeGemmParams& p, bool gated, cudaStream_t stream);
+int launch_moe_gemm(const MoeGemmParams& p, MoeForm form, cudaStream_t stream);
 // out[t] = sum over c < top of parts[t * top + c] (+ shared[t]), float32; with `chosen` the choices from
 // first_identity on count as pair_weights[t, c] * x[t].
 int launch_moe_combine(const float* parts, const void* shared, int shared_dtype, float* out, int64_t num_tokens,
                        int64_t width, int top, const int32_t* chosen, const float* pair_weights, const void* x,
                        int x_dtype, int first_identity, cudaStream_t stream);
 
-enum Activation : int { kActReluSquared = 0, kActGeluTanh = 1, kActSilu = 2 };
+enum Activation : int { kActReluSquared = 0, kActGeluTanh = 1, kActSilu = 2, kActGelu = 3, kActLast = 3 };
 int launch_activation(const void* in, void* out, int64_t total, int kind, int dtype, cudaStream_t stream);
+// the same of `width` columns of a wider matrix into columns of another
+int launch_activation_columns(const void* in, void* out, int64_t tokens, int width, int64_t in_stride, int64_t out_stride,
+                              int kind, int dtype, cudaStream_t stream);
 
 // tokens[r] = argmax(logits[r]) where temperature[r] == 0, else the inverse-CDF draw of
 // softmax(logits[r] / temperature[r]) at uniform[r].
@@ -582,6 +605,7 @@ struct SsmPrepParams {
 int launch_ssm_prep(const SsmPrepParams& p, cudaStream_t stream);
 struct ConvTailParams {
   const void* x;
+  const float* bias;           // [channels] or null: what is kept is x plus it
   int64_t x_stride;
   int conv_off, channels, taps;
   float* state;
@@ -591,6 +615,38 @@ struct ConvTailParams {
   int num_seqs, num_slots, dtype;
 };
 int launch_conv_tail(const ConvTailParams& p, cudaStream_t stream);
+
+// The q, k and v heads of one product, each channel plus its bias through a short causal convolution, q and k turned by
+// position, k and v to their cache slots (conv_prep.cu).
+struct ConvPrepParams {
+  const void* x;               // [N, x_stride]: NH * D of q, NKV * D of k, NKV * DV of v
+  int64_t x_stride;
+  const float* bias;           // [channels] or null, channels = (NH + NKV) * D + NKV * DV
+  const float* conv;           // [channels, taps], the last tap is the current token's
+  float* state;                // [slots, state_stride]; the last taps - 1 inputs [taps - 1, channels] from tail_off
+  int64_t state_stride, tail_off;
+  const int32_t* cu_q;         // [num_seqs + 1]
+  const int32_t* state_slots;  // [num_seqs], negative: a padded sequence (no inputs before it, nothing kept)
+  const int32_t* positions;    // [N]
+  const int32_t* slots;        // [N] page * page_size + offset, negative: not stored; may be null
+  const float* freq;           // [rotary_dims / 2]
+  void* q_out;                 // [N, NH * D]
+  void* k_cache;               // [num_pages, NKV, page_size, k_row_stride]
+  void* v_cache;
+  int64_t num_tokens, num_pages, k_row_stride, v_row_stride;
+  int channels, taps, num_seqs, num_slots;
+  int num_heads, num_kv_heads, head_dim, v_dim, page_size;
+  int rotary_dims, layout;     // layout 0: dim i pairs with i + rotary_dims / 2; 1: dim 2i with 2i + 1
+  float factor;                // on cos and sin
+  int keep_tail;               // 1: every sequence has one token in this step; the kernel moves the tail itself
+  int run;                     // filled in by the launcher: tokens per block
+  int dtype;
+  int* status;
+};
+int launch_conv_rotary_prep(const ConvPrepParams& p, cudaStream_t stream);
+// out[t, c] = in[t, c] * sigmoid(x[t, c]) * factor for c < width; rows of x and out lie x_stride / out_stride apart.
+int launch_gate_columns(const void* in, const void* x, void* out, int64_t tokens, int width, int64_t x_stride,
+                        int64_t out_stride, float factor, int dtype, cudaStream_t stream);
 
 // hidden[t] += table[(previous token * mul_prev + token * mul_cur) mod buckets] (row `buckets` at position 0); the
 // token before a step's first row comes from, and the step's last token goes to, last_token[slot * state_stride]
@@ -611,6 +667,41 @@ struct PairRowsParams {
 };
 int launch_pair_rows_add(const PairRowsParams& p, cudaStream_t stream);
 int launch_stream_add(float* hidden, const float* other, int64_t n, cudaStream_t stream);
+// hidden += a + b + (a token's `top` rows of parts in order) + shared, whichever are given; copy (or null) receives the
+// new rows in bfloat16 or float32.
+struct StreamSumParams {
+  float* hidden;               // [N, width]
+  const void* a;
+  const void* b;
+  int a_dtype, b_dtype;
+  const float* parts;          // [N * top, width] or null
+  int top;
+  const void* shared;
+  int shared_dtype;
+  void* copy;
+  int copy_dtype;
+  int64_t num_tokens;
+  int width;
+};
+int launch_stream_sum(const StreamSumParams& p, cudaStream_t stream);
+// out[t] = [hidden[t] | start[t]] in `dtype` (width columns each)
+int launch_stream_concat(const float* hidden, const float* start, void* out, int64_t num_tokens, int width, int dtype,
+                         cudaStream_t stream);
+// hidden[t] += row
+int launch_stream_row_add(float* hidden, const float* row, int64_t num_tokens, int width, cudaStream_t stream);
+// out[t, c] = gelu_tanh(z[t, c]) * table[token t, col_off + c]
+struct TokenGateParams {
+  const void* z;               // [N, dim]
+  const int32_t* ids;          // [N]; -(r + 1) stands for sampled[r]
+  const int32_t* sampled;
+  int64_t num_sampled;
+  const void* table;           // [vocab, table_stride]
+  void* out;                   // [N, dim]
+  int64_t num_tokens, table_stride, col_off, vocab;
+  int dim, dtype;
+  int* status;
+};
+int launch_token_gate(const TokenGateParams& p, cudaStream_t stream);
 int launch_scaled_sum(const void* a, const void* b, void* out, float sa, float sb, int64_t n, int dtype,
                       cudaStream_t stream);
 

@@ -320,9 +320,63 @@ __global__ void activation_kernel(const T* __restrict__ in, T* __restrict__ out,
   for (int64_t i = idx; i < min(idx + 8, total); ++i) out[i] = from_float<T>(activation_value(to_float<T>(in[i]), kind));
 }
 
+// out[t, c] = activation(in[t, c]) for c < width, rows in_stride / out_stride apart
+template <typename T>
+__global__ void __launch_bounds__(256) activation_columns_kernel(const T* __restrict__ in, T* __restrict__ out, int64_t total,
+                                                                 int width, int64_t in_stride, int64_t out_stride, int kind,
+                                                                 int vec) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t i = (blockIdx.x * (int64_t)blockDim.x + threadIdx.x) * (vec ? 8 : 1);
+  if (i >= total) return;
+  const int64_t token = i / width;
+  const int c = (int)(i - token * width);
+  const T* src = in + token * in_stride + c;
+  T* dst = out + token * out_stride + c;
+  if (!vec) {
+    dst[0] = from_float<T>(activation_value(to_float<T>(src[0]), kind));
+    return;
+  }
+  float v[8];
+  load8<T>(src, v);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) v[e] = activation_value(v[e], kind);
+  if constexpr (sizeof(T) == 2) {
+    uint4 packed;
+    uint32_t* w = reinterpret_cast<uint32_t*>(&packed);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const __nv_bfloat162 pair = __floats2bfloat162_rn(v[2 * e], v[2 * e + 1]);
+      w[e] = *reinterpret_cast<const uint32_t*>(&pair);
+    }
+    *reinterpret_cast<uint4*>(dst) = packed;
+  } else {
+    *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(dst + 4) = make_float4(v[4], v[5], v[6], v[7]);
+  }
+}
+
+int launch_activation_columns(const void* in, void* out, int64_t tokens, int width, int64_t in_stride, int64_t out_stride,
+                              int kind, int dtype, cudaStream_t stream) {
+  const int64_t total = tokens * width;
+  if (total == 0) return 0;
+  if (kind < kActReluSquared || kind > kActLast) return (int)cudaErrorInvalidValue;
+  const int per16 = dtype == kBFloat16 ? 8 : 4;
+  const int vec = width % 8 == 0 && in_stride % per16 == 0 && out_stride % per16 == 0 &&
+                  (reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out)) % 16 == 0;
+  const int64_t blocks = (total / (vec ? 8 : 1) + 255) / 256;
+  if (blocks > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
+  if (dtype == kBFloat16)
+    return (int)launch_chain(activation_columns_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(256), 0, stream,
+                             dim3(1, 1, 1), (const __nv_bfloat16*)in, (__nv_bfloat16*)out, total, width, in_stride,
+                             out_stride, kind, vec);
+  return (int)launch_chain(activation_columns_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, dim3(1, 1, 1),
+                           (const float*)in, (float*)out, total, width, in_stride, out_stride, kind, vec);
+}
+
 int launch_activation(const void* in, void* out, int64_t total, int kind, int dtype, cudaStream_t stream) {
   if (total == 0) return 0;
-  if (kind < kActReluSquared || kind > kActSilu) return (int)cudaErrorInvalidValue;
+  if (kind < kActReluSquared || kind > kActLast) return (int)cudaErrorInvalidValue;
   const int threads = 256;
   const int64_t blocks = ((total + 7) / 8 + threads - 1) / threads;
   if (blocks > 0x7fffffffLL) return (int)cudaErrorInvalidValue;

@@ -1,7 +1,7 @@
 // A feed-forward of routed experts, entirely on the device (no host read of the routing).
 //
 //   moe_router:   the router's logits for a few tokens (a warp per token and expert); larger steps use the library.
-//   moe_route:    per token: s = sigmoid(logits); choice = s + correction; the experts form equal groups of
+//   moe_route:    per token: s = sigmoid(logits + bias) or a softmax of them; choice = s + correction; the experts form equal groups of
 //                 neighbours, a group's score is the sum of its group_top largest choice scores, only experts of the
 //                 keep best groups can be chosen; the top largest remaining choice scores are chosen (ties: the lower
 //                 index); weights = chosen s / (their sum + eps) * scale, or chosen s * scale.  One warp per token, all
@@ -10,7 +10,8 @@
 //                 pairs in that order (within an expert in no particular order: every row is computed by itself).
 //   moe_gate_up:  for the sorted rows of every expert, both products with the expert's matrices and the clamped
 //                 activation on the output tile.
-//   moe_down:     the third product, times the pair's weight, written to the pair's own row (float32).
+//   moe_up:       the one first product of experts without a gate, with an activation on the output tile.
+//   moe_down:     the last product, times the pair's weight, written to the pair's own row (float32).
 //   moe_combine:  a token's rows added up in the order of its choices, plus the shared expert's row; choices that
 //                 are the identity (they lie behind the experts: the sort puts their pairs last and no product sees
 //                 them) count as their weight times the token's input.
@@ -49,20 +50,21 @@ __global__ void moe_route_kernel(MoeRouteParams p) {
   float* group_score = choice + E;
   float* group_kept = group_score + groups;
   const float* z = p.logits + token * E;
+  auto logit = [&](int e) -> float { return p.bias != nullptr ? z[e] + p.bias[e] : z[e]; };
   // softmax scores: the row's maximum and the sum of the exponentials first (a row of padding may hold anything)
   float row_max = 0.f, row_inv = 1.f;
   if (p.score_kind == 1) {
     float m = -FLT_MAX;
     for (int e = lane; e < E; e += 32)
-      if (z[e] == z[e]) m = fmaxf(m, fminf(z[e], FLT_MAX));
+      if (logit(e) == logit(e)) m = fmaxf(m, fminf(logit(e), FLT_MAX));
     row_max = warp_max(m);
     float sum = 0.f;
-    for (int e = lane; e < E; e += 32) sum += expf(z[e] - row_max);
+    for (int e = lane; e < E; e += 32) sum += expf(logit(e) - row_max);
     sum = warp_sum(sum);
     row_inv = 1.f / sum;
   }
   for (int e = lane; e < E; e += 32) {
-    const float s = p.score_kind == 1 ? expf(z[e] - row_max) * row_inv : 1.f / (1.f + expf(-z[e]));
+    const float s = p.score_kind == 1 ? expf(logit(e) - row_max) * row_inv : 1.f / (1.f + expf(-logit(e)));
     float c = p.correction != nullptr ? s + p.correction[e] : s;
     if (!(c == c)) c = -FLT_MAX;          // a row of padding may hold anything; the choice must still be an expert
     score[e] = s;
@@ -278,8 +280,9 @@ __device__ __forceinline__ void find_tile(const int32_t* offsets, int experts, i
 }
 }  // namespace
 
-template <typename T, bool GATED>
+template <typename T, int FORM>
 __global__ void __launch_bounds__(kGemmThreads) moe_gemm_kernel(MoeGemmParams p) {
+  constexpr bool GATED = FORM == kMoeGated, FIRST = FORM != kMoeDown;
   __shared__ float a_tile[kTileK][kTileRows + 1];
   __shared__ float w_tile[GATED ? 2 : 1][kTileK][kTileCols + 1];
   __shared__ int tile_info[3];
@@ -301,7 +304,7 @@ __global__ void __launch_bounds__(kGemmThreads) moe_gemm_kernel(MoeGemmParams p)
   if (threadIdx.x < kTileRows) {
     const int r = threadIdx.x;
     int64_t src = -1;
-    if (r < rows) src = GATED ? (int64_t)(p.order[row0 + r] / p.top) : (int64_t)(row0 + r);
+    if (r < rows) src = FIRST ? (int64_t)(p.order[row0 + r] / p.top) : (int64_t)(row0 + r);
     row_source[r] = src;
   }
   __syncthreads();
@@ -350,6 +353,13 @@ __global__ void __launch_bounds__(kGemmThreads) moe_gemm_kernel(MoeGemmParams p)
         const float g = fminf(acc[0][i][j], p.limit);
         const float u = fminf(fmaxf(acc[GATED ? 1 : 0][i][j], -p.limit), p.limit);
         dst[c] = from_float<T>(g / (1.f + expf(-p.slope * g)) * (u + p.up_offset));
+      }
+    } else if (FIRST) {
+      T* dst = (T*)p.out + (int64_t)(row0 + r) * N;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int c = col0 + tx * 4 + j;
+        if (c < N) dst[c] = from_float<T>(activation_value(acc[0][i][j], p.activation));
       }
     } else {
       const int pair = p.order[row0 + r];
@@ -415,8 +425,9 @@ __device__ __forceinline__ void find_tile_of(const int32_t* offsets, int experts
 }
 }  // namespace
 
-template <bool GATED, int BM>
+template <int FORM, int BM>
 __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(MoeGemmParams p) {
+  constexpr bool GATED = FORM == kMoeGated, FIRST = FORM != kMoeDown;
   // BM sorted rows of one expert per CTA (64, or 128 where experts have rows enough to fill such tiles: a warp then
   // holds 64 x 32 of the output and every weight fragment it fetches serves four row fragments instead of two)
   extern __shared__ __align__(16) unsigned char mma_smem[];
@@ -445,7 +456,7 @@ __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(MoeGemmParams p) {
   if (threadIdx.x < BM) {
     const int r = threadIdx.x;
     int64_t src = -1;
-    if (r < rows) src = GATED ? (int64_t)(p.order[row0 + r] / p.top) : (int64_t)(row0 + r);
+    if (r < rows) src = FIRST ? (int64_t)(p.order[row0 + r] / p.top) : (int64_t)(row0 + r);
     row_source[r] = src;
   }
   __syncthreads();
@@ -543,6 +554,16 @@ __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(MoeGemmParams p) {
             dst[c] = __float2bfloat16_rn(g / (1.f + expf(-p.slope * g)) * (u + p.up_offset));
           }
         }
+      } else if (FIRST) {
+        __nv_bfloat16* dst = (__nv_bfloat16*)p.out + (int64_t)(row0 + r) * N;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int c = col0 + wn * 32 + j * 8 + (lane & 3) * 2 + e;
+            if (c < N) dst[c] = __float2bfloat16_rn(activation_value(acc[i][j][half * 2 + e], p.activation));
+          }
+        }
       } else {
         const int pair = p.order[row0 + r];
         const float weight = p.weights[pair];
@@ -565,14 +586,14 @@ static bool moe_gemm_takes_mma(const MoeGemmParams& p) {
          (reinterpret_cast<uintptr_t>(p.a) | reinterpret_cast<uintptr_t>(p.w)) % 16 == 0;
 }
 
-template <bool GATED, int BM>
+template <int FORM, int BM>
 static int launch_moe_mma(const MoeGemmParams& p, cudaStream_t stream) {
   const int64_t row_tiles = p.pairs / BM + (p.pairs < p.experts ? p.pairs : p.experts);
-  const int cols = GATED ? kMmaWeightRows / 2 : kMmaWeightRows;
+  const int cols = FORM == kMoeGated ? kMmaWeightRows / 2 : kMmaWeightRows;
   const int64_t col_tiles = (p.n + cols - 1) / cols;
   if (row_tiles > 65535 || col_tiles > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
   const size_t smem = sizeof(__nv_bfloat16) * kMmaStages * (BM + kMmaWeightRows) * kMmaPitch;
-  auto kernel = moe_gemm_mma_kernel<GATED, BM>;
+  auto kernel = moe_gemm_mma_kernel<FORM, BM>;
   if (smem > 48 * 1024) {
     cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (err != cudaSuccess) return (int)err;
@@ -598,8 +619,9 @@ __device__ __forceinline__ void unpack8(const uint4& raw, float (&v)[8]) {
 }
 }  // namespace
 
-template <bool GATED>
+template <int FORM>
 __global__ void __launch_bounds__(kGemvWarps * 32) moe_gemv_kernel(MoeGemmParams p) {
+  constexpr bool GATED = FORM == kMoeGated, FIRST = FORM != kMoeDown;
   pdl_launch_dependents();
   pdl_wait();
   const int expert = blockIdx.y;
@@ -618,7 +640,7 @@ __global__ void __launch_bounds__(kGemvWarps * 32) moe_gemv_kernel(MoeGemmParams
     for (int r = 0; r < kGemvRows; ++r) {
       const int sorted = begin + r0 + min(r, count - 1);        // rows beyond the group repeat its last one, unused
       pair[r] = p.order[sorted];
-      const int64_t src = GATED ? (int64_t)(pair[r] / p.top) : (int64_t)sorted;
+      const int64_t src = FIRST ? (int64_t)(pair[r] / p.top) : (int64_t)sorted;
       x[r] = reinterpret_cast<const uint4*>(a + src * K);
     }
     for (int f = 0; f < kPerWarp; ++f) {
@@ -662,6 +684,9 @@ __global__ void __launch_bounds__(kGemvWarps * 32) moe_gemv_kernel(MoeGemmParams
           const float u = fminf(fmaxf(second, -p.limit), p.limit);
           ((__nv_bfloat16*)p.out)[(int64_t)(begin + r0 + lane) * N + feature] =
               __float2bfloat16_rn(g / (1.f + expf(-p.slope * g)) * (u + p.up_offset));
+        } else if (FIRST) {
+          ((__nv_bfloat16*)p.out)[(int64_t)(begin + r0 + lane) * N + feature] =
+              __float2bfloat16_rn(activation_value(first, p.activation));
         } else {
           int mine = pair[0];
 #pragma unroll
@@ -674,18 +699,17 @@ __global__ void __launch_bounds__(kGemvWarps * 32) moe_gemv_kernel(MoeGemmParams
   }
 }
 
-int launch_moe_gemm(const MoeGemmParams& p, bool gated, cudaStream_t stream) {
-  if (p.pairs == 0) return 0;
-  if (p.experts <= 0 || p.experts > kMoeMaxExperts || p.k <= 0 || p.n <= 0 || p.top <= 0) return (int)cudaErrorInvalidValue;
+namespace {
+template <int FORM>
+int launch_moe_form(const MoeGemmParams& p, cudaStream_t stream) {
   // 0: by size; 1: float arithmetic; 2: mma.sync tiles; 3: the few-rows form
   const bool tensor_ok = moe_gemm_takes_mma(p);
   if ((p.force_plain == 2 || p.force_plain == 3) && !tensor_ok) return (int)cudaErrorInvalidValue;
-  if (p.force_plain == 3 || (p.force_plain == 0 && tensor_ok && gated && p.pairs <= kMoeFewRowPairs)) {
+  if (p.force_plain == 3 || (p.force_plain == 0 && tensor_ok && FORM != kMoeDown && p.pairs <= kMoeFewRowPairs)) {
     const int64_t col_tiles = (p.n + kGemvFeatures - 1) / kGemvFeatures;
     if (col_tiles > 0x7fffffffLL || p.experts > 65535) return (int)cudaErrorInvalidValue;
     const dim3 grid((unsigned)col_tiles, (unsigned)p.experts);
-    if (gated) return (int)launch_chain(moe_gemv_kernel<true>, grid, dim3(kGemvWarps * 32), 0, stream, dim3(1, 1, 1), p);
-    return (int)launch_chain(moe_gemv_kernel<false>, grid, dim3(kGemvWarps * 32), 0, stream, dim3(1, 1, 1), p);
+    return (int)launch_chain(moe_gemv_kernel<FORM>, grid, dim3(kGemvWarps * 32), 0, stream, dim3(1, 1, 1), p);
   }
   if (tensor_ok && p.force_plain != 1) {
     // tiles of 128 rows where the experts' runs are long enough to fill them.  Measured (gated / down product, us):
@@ -695,21 +719,29 @@ int launch_moe_gemm(const MoeGemmParams& p, bool gated, cudaStream_t stream) {
       const char* v = getenv("AKV_MOE_TALL_ROWS");
       return v != nullptr && v[0] != '\0' ? (int64_t)atoll(v) : (int64_t)384;
     }();
-    const bool tall = p.pairs >= tall_rows * p.experts;
-    if (gated) return tall ? launch_moe_mma<true, 128>(p, stream) : launch_moe_mma<true, 64>(p, stream);
-    return tall ? launch_moe_mma<false, 128>(p, stream) : launch_moe_mma<false, 64>(p, stream);
+    return p.pairs >= tall_rows * p.experts ? launch_moe_mma<FORM, 128>(p, stream) : launch_moe_mma<FORM, 64>(p, stream);
   }
   // every expert may end in a tile that is not full
   const int64_t row_tiles = p.pairs / kTileRows + (p.pairs < p.experts ? p.pairs : p.experts);
   const int64_t col_tiles = (p.n + kTileCols - 1) / kTileCols;
   if (row_tiles > 65535 || col_tiles > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
   const dim3 grid((unsigned)col_tiles, (unsigned)row_tiles);
-  if (p.dtype == kBFloat16) {
-    if (gated) return (int)launch_chain(moe_gemm_kernel<__nv_bfloat16, true>, grid, dim3(kGemmThreads), 0, stream, dim3(1, 1, 1), p);
-    return (int)launch_chain(moe_gemm_kernel<__nv_bfloat16, false>, grid, dim3(kGemmThreads), 0, stream, dim3(1, 1, 1), p);
+  if (p.dtype == kBFloat16)
+    return (int)launch_chain(moe_gemm_kernel<__nv_bfloat16, FORM>, grid, dim3(kGemmThreads), 0, stream, dim3(1, 1, 1), p);
+  return (int)launch_chain(moe_gemm_kernel<float, FORM>, grid, dim3(kGemmThreads), 0, stream, dim3(1, 1, 1), p);
+}
+}  // namespace
+
+int launch_moe_gemm(const MoeGemmParams& p, MoeForm form, cudaStream_t stream) {
+  if (p.pairs == 0) return 0;
+  if (p.experts <= 0 || p.experts > kMoeMaxExperts || p.k <= 0 || p.n <= 0 || p.top <= 0) return (int)cudaErrorInvalidValue;
+  switch (form) {
+    case kMoeGated: return launch_moe_form<kMoeGated>(p, stream);
+    case kMoeUp:
+      if (p.activation < 0 || p.activation > kActLast) return (int)cudaErrorInvalidValue;
+      return launch_moe_form<kMoeUp>(p, stream);
+    default: return launch_moe_form<kMoeDown>(p, stream);
   }
-  if (gated) return (int)launch_chain(moe_gemm_kernel<float, true>, grid, dim3(kGemmThreads), 0, stream, dim3(1, 1, 1), p);
-  return (int)launch_chain(moe_gemm_kernel<float, false>, grid, dim3(kGemmThreads), 0, stream, dim3(1, 1, 1), p);
 }
 
 template <typename TS>

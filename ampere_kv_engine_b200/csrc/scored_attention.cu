@@ -9,6 +9,8 @@
 //                 with keep_first > 0 the keys j < keep_first stay visible behind a window (at their true positions)
 //   out_i = softmax over the visible j of score(i, j) applied to v_j, times gate[i, h] (if given), times out_scale
 //   sigmoid_weights: the weight of a visible key is sigmoid(score + head_bias[h]) instead, not normalised over keys
+//   sink: the softmax's denominator also counts exp(sink[h]): the first split starts from the maximum sink[h] and the
+//         sum 1, as if a key of that score and of value zero had come first
 //
 // Keys are rows of `head_dim` elements, values rows of `v_dim`; both live in paged storage
 // [pages, kv heads, page size, row stride] whose row strides are given, so a value may be a
@@ -106,6 +108,10 @@ scored_attention_kernel(ScoredAttentionParams sp, int row_groups, int64_t total_
   for (int r = 0; r < R; ++r) {
     m[r] = -CUDART_INF_F;
     l[r] = 0.f;
+    if (sp.sink != nullptr && split == 0 && r < nrows) {
+      m[r] = sp.sink[kvh * G + (row0 + r) % G];
+      l[r] = lane == 0 ? 1.f : 0.f;
+    }
 #pragma unroll
     for (int c = 0; c < DC; ++c) acc[r][c] = 0.f;
   }
@@ -356,7 +362,8 @@ int launch_scored_attention(const ScoredAttentionParams& sp, cudaStream_t stream
   if (p.head_dim < 1 || sp.v_dim < 1 || sp.v_dim > 512 || p.num_heads % p.num_kv_heads || p.num_splits < 1 ||
       p.num_splits > kMergeSplits ||
       sp.k_row_stride < p.head_dim || sp.v_row_stride < sp.v_dim || sp.chunk < 0 || sp.softcap < 0.f ||
-      sp.keep_first < 0 || (sp.keep_first > 0 && (p.window <= 0 || sp.chunk > 0)))
+      sp.keep_first < 0 || (sp.keep_first > 0 && (p.window <= 0 || sp.chunk > 0)) ||
+      (sp.sink != nullptr && sp.sigmoid_weights))
     return (int)cudaErrorInvalidValue;
   // kept first keys, weights without a softmax and an output factor: the tcgen05 prompt kernel, the tensor-core
   // kernel for single tokens and the general kernel

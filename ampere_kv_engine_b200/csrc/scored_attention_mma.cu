@@ -167,6 +167,17 @@ scored_attention_mma_kernel(ScoredAttentionParams sp, int row_groups, int ldk) {
   };
 
   float m[2] = {-CUDART_INF_F, -CUDART_INF_F}, l[2] = {0.f, 0.f};      // m in log2 units
+  // a sink: the walk of the first split starts as if a key of that score and of value zero had come first (every warp
+  // holds the maximum, one lane of the CTA counts the one)
+  if (sp.sink != nullptr && split == 0) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      if (g + 8 * r < nrows) {
+        m[r] = sp.sink[kvh * G + (row0 + g + 8 * r) % G] * kLog2eF;
+        l[r] = (warp == 0 && (lane & 3) == 0) ? 1.f : 0.f;
+      }
+    }
+  }
   float o[NV][4];
 #pragma unroll
   for (int v = 0; v < NV; ++v) o[v][0] = o[v][1] = o[v][2] = o[v][3] = 0.f;

@@ -10,7 +10,7 @@
 //               so that with q = C, k = B, v = dt x the recurrence S <- decay S + k v^T, o = S^T q is the scan's
 //               per-token-decay mode with H / G heads sharing a q and k.
 //   conv_tail:  moves each sequence's last taps - 1 inputs of the convolved channels into the state slot; a thread per
-//               (sequence, channel) reads all it needs before it writes.
+//               (sequence, channel) reads all it needs before it writes.  A bias per channel may belong to the inputs.
 //
 // Everything after the product is float32.  A sequence whose state slot is negative (padding of a captured step) is
 // left alone and its rows are zero.
@@ -92,6 +92,7 @@ __global__ void __launch_bounds__(128) conv_tail_kernel(ConvTailParams p, int ch
   if (c >= p.channels || n <= 0 || slot < 0 || slot >= p.num_slots) return;
   const int keep = p.taps - 1;
   const T* x = (const T*)p.x;
+  const float bias = p.bias != nullptr ? p.bias[c] : 0.f;
   float* before = p.state + (int64_t)slot * p.state_stride + p.tail_off;
   float kept[kConvMaxTaps - 1];
 #pragma unroll
@@ -99,7 +100,7 @@ __global__ void __launch_bounds__(128) conv_tail_kernel(ConvTailParams p, int ch
     kept[i] = 0.f;
     if (i < keep) {
       const int back = n - keep + i;          // index within the step's tokens of this sequence
-      kept[i] = back >= 0 ? to_float<T>(x[(first + back) * p.x_stride + p.conv_off + c])
+      kept[i] = back >= 0 ? to_float<T>(x[(first + back) * p.x_stride + p.conv_off + c]) + bias
                           : before[(int64_t)(i + n) * p.channels + c];
     }
   }

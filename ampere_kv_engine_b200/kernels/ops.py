@@ -417,13 +417,15 @@ def choose_splits_shared_rows(num_tiles: int, num_kv_heads: int, rows_per_tile: 
 def scored_attention(q, k_cache, v_cache, block_table, cu_q, ctx_lens, tile_seq, tile_q0, tile_nq, *, num_tiles,
                      q_tile, num_splits, num_heads, num_kv_heads, v_dim, scale, window=0, chunk=0, softcap=0.0,
                      slopes=None, gate=None, partials=None, status=None, out=None, kernel: str = "auto",
-                     keep_first: int = 0, sigmoid_weights: bool = False, head_bias=None, out_scale: float = 1.0):
+                     keep_first: int = 0, sigmoid_weights: bool = False, head_bias=None, out_scale: float = 1.0,
+                     sink=None):
     """Causal attention of the batch's new tokens over paged keys and values of different widths, with the score
     reshaped before the softmax: ``softcap * tanh(score / softcap)`` (``softcap`` > 0), less ``slopes[h]`` times the
     distance to the key (``slopes`` float32 [heads]); a query sees the last ``window`` keys (``window`` > 0) of its own
     block of ``chunk`` positions (``chunk`` > 0), and with ``keep_first`` the keys at positions below it behind the
     window too; ``gate`` (float32 [tokens, heads]) scales each head's output and ``out_scale`` all of them.  With
-    ``sigmoid_weights`` there is no softmax: a visible key weighs ``sigmoid(score + head_bias[h])``.
+    ``sigmoid_weights`` there is no softmax: a visible key weighs ``sigmoid(score + head_bias[h])``.  ``sink`` (float32
+    [heads]): the softmax's denominator also counts ``exp(sink[h])``, which belongs to no key.
     ``k_cache`` / ``v_cache``: [pages, kv heads, page size, width]; they may be one tensor whose rows are read whole
     as keys and in their first ``v_dim`` elements as values.  Returns [tokens, heads * v_dim]; only the rows of the
     given tiles are written.  ``kernel``: ``"auto"`` takes the tensor-core kernels where they fit
@@ -437,7 +439,7 @@ def scored_attention(q, k_cache, v_cache, block_table, cu_q, ctx_lens, tile_seq,
                            num_tiles, q_tile, num_splits, num_heads, num_kv_heads, int(v_dim), int(window or 0),
                            int(chunk or 0), float(scale), float(softcap or 0.0), slopes, gate, status,
                            {"auto": 0, "general": 1}[kernel], int(keep_first or 0), bool(sigmoid_weights), head_bias,
-                           float(out_scale))
+                           float(out_scale), **({} if sink is None else {"sink": sink}))
     _launched(2 if num_splits > 1 else 1)
     return out
 
@@ -494,7 +496,7 @@ def rotate_pairs(x, out, positions, inv_freq, *, heads, cols, rotary_dims, in_of
     _launched()
 
 
-ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2}
+ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "gelu": 3}
 
 
 def linear_activation(x, weight: torch.Tensor, kind: str, status: torch.Tensor | None = None) -> torch.Tensor:
@@ -508,9 +510,20 @@ def linear_activation(x, weight: torch.Tensor, kind: str, status: torch.Tensor |
 
 
 def activation(x: torch.Tensor, kind: str) -> torch.Tensor:
-    """``relu(x) ** 2`` (``"relu2"``), the tanh form of GELU (``"gelu_tanh"``) or SiLU, element by element."""
+    """``relu(x) ** 2`` (``"relu2"``), the tanh form of GELU (``"gelu_tanh"``), SiLU (``"silu"``) or GELU itself
+    (``"gelu"``), element by element."""
     out = torch.empty_like(x)
     ext().activation(x, out, ACTIVATIONS[kind])
+    _launched()
+    return out
+
+
+def activation_columns(x: torch.Tensor, off: int, width: int, kind: str, out=None, out_off: int = 0) -> torch.Tensor:
+    """:func:`activation` of the columns ``[off, off + width)`` of ``x``; with ``out`` (a wider matrix) written to its
+    columns from ``out_off`` on."""
+    if out is None:
+        out, out_off = torch.empty((x.shape[0], width), dtype=x.dtype, device=x.device), 0
+    ext().activation_columns(x, int(off), int(width), ACTIVATIONS[kind], out, int(out_off))
     _launched()
     return out
 
@@ -548,36 +561,54 @@ def delta_state_floats(num_heads: int, num_kv_heads: int, head_dim: int, v_dim: 
 
 
 def delta_prep(x, conv, rate_log, step_bias, state, cu_q, state_slots, *, num_heads, num_kv_heads, head_dim, v_dim,
-               taps, unit_eps):
+               taps, unit_eps, steps=None, step_off: int = 0, channel_decay: bool = False, x_off: int = 0,
+               beta_off: int = 0):
     """From one product ``x`` [tokens, q | k | v | gate | beta | step] (``num_kv_heads`` heads of ``head_dim`` for q
     and k, ``num_heads`` of ``v_dim`` for v and gate, a column per head for beta and step): q, k and v through their
     causal convolutions over the sequence's own earlier tokens (``conv`` float32 [channels, taps], last tap the
     current token's; before the step's first token the inputs come from ``state[slot, memory:]``, zeros at a
     sequence's start) and SiLU; q and k scaled to unit length (q also by ``head_dim ** -0.5``);
     ``beta = sigmoid(.)``, ``decay = exp(-exp(rate_log) * softplus(step + step_bias))``.  ``cu_q`` [sequences + 1]
-    gives each sequence's rows, ``state_slots`` its slot (negative: a padded sequence, left alone).  Returns
-    (float32 [tokens, q | k | v], float32 [tokens, beta per head | decay per head]).  The state is not changed."""
+    gives each sequence's rows, ``state_slots`` its slot (negative: a padded sequence, left alone).  With ``steps``
+    (a product of its own, float32 or the compute dtype) the step columns stand there from ``step_off`` on, and ``x`` is
+    any matrix that holds [q | k | v] from ``x_off`` and the beta columns from ``beta_off``; with ``channel_decay`` there
+    are ``num_heads * head_dim`` steps and decays (``step_bias`` likewise).  Returns
+    (float32 [tokens, q | k | v], float32 [tokens, beta per head | decays]).  The state is not changed."""
     n = x.shape[0]
     channels = 2 * num_kv_heads * head_dim + num_heads * v_dim
     qkv = torch.empty((n, channels), dtype=torch.float32, device=x.device)
-    coef = torch.empty((n, 2 * num_heads), dtype=torch.float32, device=x.device)
+    coef = torch.empty((n, num_heads * (1 + (head_dim if channel_decay else 1))), dtype=torch.float32, device=x.device)
+    extra = {} if steps is None else dict(steps=steps, step_off=int(step_off), channel_decay=bool(channel_decay),
+                                          x_off=int(x_off), beta_off=int(beta_off))
     ext().delta_prep(x, conv, rate_log, step_bias, state, cu_q, state_slots, qkv, coef, num_heads, num_kv_heads,
-                     head_dim, v_dim, taps, float(unit_eps))
+                     head_dim, v_dim, taps, float(unit_eps), **extra)
     _launched()
     return qkv, coef
 
 
+DELTA_GATES = {"silu": 0, "sigmoid": 1}
+
+
 def delta_scan(qkv, coef, x, norm_weight, state, cu_q, state_slots, *, num_heads, num_kv_heads, head_dim, v_dim, taps,
-               norm_eps):
+               norm_eps, gates=None, gate_off: int = 0, gate: str = "silu", channel_decay: bool = False, x_off: int = 0,
+               factor: float = 1.0, out=None, out_off: int = 0):
     """The recurrence over the step's tokens, sequence by sequence and head by head, from and into ``state``
     [slots, delta_state_floats(...)[1]] float32: ``S *= decay; u = beta (v - S^T k);
     S += k u^T; o = S^T q``; then ``o / sqrt(mean(o^2) + norm_eps) * norm_weight * silu(gate)`` with the gate columns
     of ``x``.  Also moves the sequence's last ``taps - 1`` convolution inputs (columns of ``x``) into the state.
-    Returns [tokens, heads * v_dim] in the dtype of ``x``."""
-    out = torch.empty((x.shape[0], num_heads * v_dim), dtype=x.dtype, device=x.device)
+    With ``gates`` (a product of its own) the gate columns stand there from ``gate_off`` on and ``x`` holds [q | k | v]
+    from ``x_off``; ``gate`` names the gate's function; ``channel_decay``: every row of S has its own decay; the result
+    is multiplied by ``factor``.  Returns [tokens, heads * v_dim] in the dtype of ``x``; with ``out`` (a wider matrix)
+    it is written to that one's columns from ``out_off`` on."""
+    if out is None:
+        out, out_off = torch.empty((x.shape[0], num_heads * v_dim), dtype=x.dtype, device=x.device), 0
     scratch = torch.empty((x.shape[0], num_heads * v_dim), dtype=torch.float32, device=x.device)
+    extra = {}
+    if gates is not None or gate != "silu" or channel_decay or factor != 1.0 or out_off or out.shape[1] != scratch.shape[1]:
+        extra = dict(gates=gates, gate_off=int(gate_off), gate_kind=DELTA_GATES[gate], channel_decay=bool(channel_decay),
+                     x_off=int(x_off), out_off=int(out_off), factor=float(factor))
     ext().delta_scan(qkv, coef, x, norm_weight, state, cu_q, state_slots, scratch, out, num_heads, num_kv_heads,
-                     head_dim, v_dim, taps, float(norm_eps))
+                     head_dim, v_dim, taps, float(norm_eps), **extra)
     _launched(2)        # the scan; the output norm and the convolutions' memory
     return out
 
@@ -608,9 +639,9 @@ MOE_SCORES = {"sigmoid": 0, "softmax": 1}
 
 
 def moe_route(logits, correction, *, top, groups, keep_groups, group_top, scale, weight_eps, score: str = "sigmoid",
-              normalize: bool = True):
+              normalize: bool = True, bias=None):
     """Scores ``sigmoid(logits)``, or with ``score="softmax"`` the softmax over all experts (float32
-    [tokens, experts]); choice scores are the scores plus ``correction``
+    [tokens, experts]), of the logits plus ``bias`` (float32 [experts] or None); choice scores are the scores plus ``correction``
     (float32 [experts] or None); experts form ``groups`` equal runs, a group's score is the sum of its ``group_top``
     largest choice scores, experts outside the ``keep_groups`` best groups cannot be chosen; the ``top`` largest
     remaining choice scores are chosen (ties: the lower index).  Returns (int32 [tokens, top], float32 [tokens, top]:
@@ -619,7 +650,7 @@ def moe_route(logits, correction, *, top, groups, keep_groups, group_top, scale,
     chosen = torch.empty((n, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((n, top), dtype=torch.float32, device=logits.device)
     ext().moe_route(logits, correction, chosen, weights, groups, keep_groups, group_top, float(scale), float(weight_eps),
-                    MOE_SCORES[score], bool(normalize))
+                    MOE_SCORES[score], bool(normalize), **({} if bias is None else {"bias": bias}))
     _launched()
     return chosen, weights
 
@@ -647,6 +678,16 @@ def moe_gate_up(x, w_gate_up, order, offsets, *, top, limit, slope, kernel: str 
     act = torch.empty((order.numel(), inter), dtype=x.dtype, device=x.device)
     ext().moe_gate_up(x, w_gate_up, order, offsets, act, top, float(limit), float(slope), MOE_FORMS[kernel],
                       float(up_offset))
+    _launched()
+    return act
+
+
+def moe_up(x, w_up, order, offsets, *, top, activation: str, kernel: str = "auto"):
+    """Row r of the result belongs to pair ``order[r]`` and is ``activation(W_up x)`` of its expert (one without a gate)
+    for the pair's token; ``w_up`` [experts, intermediate, hidden].  [tokens * top, intermediate] in the dtype of ``x``.
+    ``kernel`` as for :func:`moe_gate_up`."""
+    act = torch.empty((order.numel(), w_up.shape[1]), dtype=x.dtype, device=x.device)
+    ext().moe_up(x, w_up, order, offsets, act, top, ACTIVATIONS[activation], MOE_FORMS[kernel])
     _launched()
     return act
 
@@ -815,7 +856,8 @@ def linear_into_residual(x: torch.Tensor, weight: torch.Tensor, hidden: torch.Te
 
 def _takes_small_m(x: torch.Tensor, weight: torch.Tensor) -> bool:
     return (use_small_m_gemm and x.is_cuda and x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16
-            and x.dim() == 2 and x.shape[0] <= SMALL_M_LIMIT and x.is_contiguous() and weight.is_contiguous()
+            and x.dim() == 2 and x.shape[0] <= SMALL_M_LIMIT and weight.is_contiguous()
+            and (x.is_contiguous() or (x.stride(1) == 1 and x.stride(0) % 8 == 0 and x.stride(0) >= x.shape[1]))
             and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0
             and ext().small_m_gemm_supported(x.shape[0], weight.shape[0], weight.shape[1]))
 
@@ -1003,6 +1045,75 @@ def stream_add(hidden: torch.Tensor, other: torch.Tensor, delta=None):
     return delta
 
 
+def stream_sum(hidden: torch.Tensor, pending, copy_dtype=None) -> torch.Tensor | None:
+    """Everything in ``pending`` (branch results in any of the forms a block may leave: tensors, stacks of partial sums,
+    an :class:`ExpertParts`, a :class:`NormedBranch`, queued products, records of sums the stream holds already) added to
+    the float32 stream ``hidden`` in place.  With ``copy_dtype`` the new stream is also returned in that dtype (the
+    stream itself when that is float32)."""
+    dense, parts = [], None
+    for p in pending:
+        if p is None or isinstance(p, (Summed, Mirrored)):
+            continue
+        if isinstance(p, PendingPhases):
+            p.launch()
+        elif isinstance(p, NormedBranch):
+            p.apply(hidden)
+        elif isinstance(p, ExpertParts):
+            if parts is None and p.identity is None:
+                parts = p
+            else:
+                dense.append(p.materialize())
+        else:
+            dense.append(p.sum(0) if p.dim() == 3 else p)
+    copy = None
+    if copy_dtype is not None and copy_dtype != torch.float32:
+        copy = torch.empty(hidden.shape, dtype=copy_dtype, device=hidden.device)
+    while len(dense) > 2:
+        ext().stream_sum(hidden, dense.pop(), dense.pop(), None, None, 0, None)
+        _launched()
+    if dense or parts is not None or copy is not None:
+        a, b = (dense + [None, None])[:2]
+        ext().stream_sum(hidden, a, b, None if parts is None else parts.parts, None if parts is None else parts.shared,
+                         0 if parts is None else parts.top, copy)
+        _launched()
+    if copy_dtype is None:
+        return None
+    return hidden if copy is None else copy
+
+
+def stream_concat(hidden: torch.Tensor, start: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+    """``[hidden | start]`` of two float32 streams [tokens, width], in ``dtype``."""
+    out = torch.empty((hidden.shape[0], 2 * hidden.shape[1]), dtype=dtype, device=hidden.device)
+    ext().stream_concat(hidden, start, out)
+    _launched()
+    return out
+
+
+def stream_row_add(hidden: torch.Tensor, row: torch.Tensor) -> torch.Tensor:
+    """``row`` (float32 [width]) added to every row of the stream in place."""
+    ext().stream_row_add(hidden, row)
+    _launched()
+    return hidden
+
+
+def token_gate(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, col_off: int, sampled=None, status=None):
+    """``gelu_tanh(z[t]) * table[id of token t, col_off : col_off + dim]`` (ids as for :func:`embedding`)."""
+    out = torch.empty_like(z)
+    ext().token_gate(z, ids, sampled, table, int(col_off), out, status)
+    _launched()
+    return out
+
+
+def gate_columns(values: torch.Tensor, x: torch.Tensor, gate_off: int, factor: float = 1.0, out=None, out_off: int = 0):
+    """``values * sigmoid(x[:, gate_off + column]) * factor``; with ``out`` (a wider matrix) written to its columns from
+    ``out_off`` on."""
+    if out is None:
+        out, out_off = torch.empty_like(values), 0
+    ext().gate_columns(values, x, int(gate_off), out, int(out_off), float(factor))
+    _launched()
+    return out
+
+
 def scaled_sum(a: torch.Tensor, b: torch.Tensor, sa: float, sb: float) -> torch.Tensor:
     """``a * sa + b * sb`` of two branch outputs, formed in float32 and rounded once to their dtype."""
     out = torch.empty_like(a)
@@ -1044,6 +1155,28 @@ def rotary_prep(x, positions, slots, freq, k_cache, v_cache, *, num_heads, num_k
                       int(rotary_dims), ROTARY_LAYOUTS[layout], float(factor), bool(value_from_key), bool(value_norm),
                       float(eps), status, q_norm, k_norm, float(row_norm_eps), int(x_off))
     _launched()
+    return q_out
+
+
+def conv_rotary_prep(x, conv, positions, slots, freq, k_cache, v_cache, state, cu_q, state_slots, *, num_heads,
+                     num_kv_heads, head_dim, v_dim, taps, rotary_dims, layout: str, factor: float = 1.0, bias=None,
+                     x_off: int = 0, tail_off: int = 0, status=None) -> torch.Tensor:
+    """From one product ``x`` whose columns from ``x_off`` hold ``[q heads | k heads | v heads]``: every channel plus its
+    ``bias`` (float32 [channels] or None), through its causal convolution over the sequence's own earlier tokens
+    (``conv`` float32 [channels, taps], last tap the current token's; before the step's first token the inputs come from
+    ``state[slot, tail_off:]``, zeros at a sequence's start); q and k turned as in :func:`rotary_prep`; k and v written
+    to their cache slots; the sequences' last ``taps - 1`` inputs left in the state.  Returns q
+    [tokens, heads * head_dim]."""
+    n, seqs = x.shape[0], cu_q.numel() - 1
+    q_out = torch.empty((n, num_heads * head_dim), dtype=x.dtype, device=x.device)
+    keep_tail = n == seqs           # a token per sequence: the same kernel moves the inputs along
+    ext().conv_rotary_prep(x, int(x_off), bias, conv, state, int(tail_off), cu_q, state_slots, positions, slots, freq, q_out,
+                           k_cache, v_cache, num_heads, num_kv_heads, head_dim, v_dim, int(taps), int(rotary_dims),
+                           ROTARY_LAYOUTS[layout], float(factor), keep_tail, status)
+    _launched()
+    if not keep_tail:
+        conv_tail(x, state, cu_q, state_slots, tail_off=tail_off, conv_off=x_off,
+                  channels=(num_heads + num_kv_heads) * head_dim + num_kv_heads * v_dim, taps=taps, bias=bias)
     return q_out
 
 
@@ -1160,12 +1293,13 @@ def ssm_prep(x, conv, conv_bias, step_bias, rate_log, state, cu_q, state_slots, 
     return out
 
 
-def conv_tail(x, state, cu_q, state_slots, *, tail_off: int, conv_off: int, channels: int, taps: int) -> None:
-    """Every sequence's last ``taps - 1`` rows of the columns ``[conv_off, conv_off + channels)`` of ``x`` (older rows
-    from what the slot held) into ``state[slot, tail_off:]`` as [taps - 1, channels]."""
+def conv_tail(x, state, cu_q, state_slots, *, tail_off: int, conv_off: int, channels: int, taps: int, bias=None) -> None:
+    """Every sequence's last ``taps - 1`` rows of the columns ``[conv_off, conv_off + channels)`` of ``x``, plus ``bias``
+    (float32 [channels] or None) (older rows from what the slot held), into ``state[slot, tail_off:]`` as [taps - 1, channels]."""
     if taps <= 1:
         return
-    ext().conv_tail(x, state, int(tail_off), cu_q, state_slots, int(conv_off), int(channels), int(taps))
+    ext().conv_tail(x, state, int(tail_off), cu_q, state_slots, int(conv_off), int(channels), int(taps),
+                    **({} if bias is None else {"bias": bias}))
     _launched()
 
 

@@ -17,8 +17,8 @@ from ..config.spec import ModelSpec
 from ..kernels import ops
 from ..parts import (attention, block, embedding, feed_forward, gated_delta, hyper, latent_attention,  # noqa: F401
                      linear_memory, norm, parallel, position, rotary_attention, routed_experts,
-                     scored_attention, state_space)             # (importing them registers the built-in kinds)
-from ..parts.base import BLOCKS, EMBEDDINGS, HEADS, NORMS, Block, CacheSpec, ParamSpec, build_part
+                     scored_attention, state_space, stream_update)   # (importing them registers the built-in kinds)
+from ..parts.base import BLOCKS, EMBEDDINGS, HEADS, NORMS, STREAM_UPDATES, Block, CacheSpec, ParamSpec, build_part
 
 
 class DecoderModel:
@@ -32,6 +32,7 @@ class DecoderModel:
         kw = dict(hidden_size=spec.hidden_size, dtype=dtype, device=self.device)
         self.embedding = build_part(EMBEDDINGS, spec.embedding, **kw)
         self.blocks = [BLOCKS.get(layer.block)(layer, **kw) for layer in spec.layers]
+        self.walk_entry = None if spec.walk_entry is None else build_part(STREAM_UPDATES, spec.walk_entry, **kw)
         self.final_norm = build_part(NORMS, spec.final_norm, **kw)
         self.head = build_part(HEADS, spec.head, **kw)
         self.loaded = False
@@ -48,6 +49,8 @@ class DecoderModel:
         for blk in self.blocks:
             for part in blk.parts():
                 yield from walk(part)
+        if self.walk_entry is not None:
+            yield from walk(self.walk_entry)
         yield from walk(self.final_norm)
         yield from walk(self.head)
 
@@ -123,14 +126,19 @@ class DecoderModel:
             hidden = self.embedding.forward(ctx.token_ids, ctx, cache=cache_views[positions])
         else:
             hidden = self.embedding.forward(ctx.token_ids, ctx)
-        # a schedule that sends the stream through layers again adds the embedding's output before each such pass
-        start = hidden.clone() if any(e.add_embedding for e in self.spec.schedule) else None
+        # a schedule that sends the stream through layers again adds the embedding's output before each such pass, or
+        # gives it to what stands before a pass
+        start = None
+        if any(e.add_embedding or e.begins_walk is not None for e in self.spec.schedule):
+            start = hidden.clone()
         delta = None
         if self.spec.streams:
             hidden = ops.hyper_expand(hidden, self.spec.streams)
         for pos, entry in enumerate(self.spec.schedule):
             if entry.add_embedding:
                 delta = ops.stream_add(hidden, start, delta)
+            if entry.begins_walk is not None:
+                hidden, delta = self.walk_entry.forward(hidden, [delta], ctx, start=start, walk=entry.begins_walk)
             hidden, delta = self.blocks[entry.layer].forward(hidden, delta, ctx, cache_views[pos])
         if ctx.num_logit_rows == 0:
             return None

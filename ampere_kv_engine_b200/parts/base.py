@@ -6,8 +6,9 @@ computes on the flat token batch of one step.  Parts never look at a model confi
 and do not know which architecture uses them; the reference, by contrast, wires one model's
 attribute paths into every function (ampere_kv/runner.py:60-77, 102-179).
 
-Kinds are looked up in eight registries (mixers, feed-forwards, norms, position encodings,
-blocks, embeddings, heads, and the connections between a sublayer and a stream kept in several copies).  Registering a new kind is one decorator call and needs no change
+Kinds are looked up in nine registries (mixers, feed-forwards, norms, position encodings,
+blocks, embeddings, heads, the connections between a sublayer and a stream kept in several copies, and the updates of the
+stream that stand between branches or between layers).  Registering a new kind is one decorator call and needs no change
 here.
 """
 
@@ -22,6 +23,9 @@ from ..config.spec import LayerSpec, PartSpec
 from ..kernels import ops
 
 
+FREE_SIZE = -1
+
+
 @dataclass(frozen=True)
 class ParamSpec:
     """One tensor a part wants from the checkpoint.
@@ -31,11 +35,20 @@ class ParamSpec:
     stored in 32-bit stays 32-bit) or ``"table"`` (integer tables, int32).  ``init`` names the random draw of the random-weights mode.
     """
 
+    #: a size of ``FREE_SIZE`` is whatever the checkpoint holds (the configuration does not say it)
     shape: tuple[int, ...]
     kind: str = "matrix"
     #: "normal": N(0, 0.02); "norm": 1 + N(0, 0.1); "around_zero": N(0, 0.1); "unit_interval": U(0, 1); "zeros"
     init: str = "normal"
     optional: bool = False
+    #: the size that random weights give a free dimension
+    free_size: int = 0
+
+    def accepts(self, shape) -> bool:
+        return len(shape) == len(self.shape) and all(w in (FREE_SIZE, g) for w, g in zip(self.shape, shape))
+
+    def drawn_shape(self) -> tuple[int, ...]:
+        return tuple(self.free_size if w == FREE_SIZE else w for w in self.shape)
 
 
 @dataclass(frozen=True)
@@ -210,6 +223,17 @@ class Connection(Part):
         raise NotImplementedError
 
 
+class StreamUpdate(Part):
+    """What happens to the residual stream itself, beside what the branches add to it: right after a layer's branches, or
+    right before a pass through a run of layers."""
+
+    def forward(self, hidden: torch.Tensor, pending: list, ctx, *, start: torch.Tensor | None = None, walk: int = 0):
+        """``pending``: results that are not yet in the stream ``hidden`` (``ops.stream_sum`` takes every form).
+        ``start``: the embedding's output, and ``walk``: the number of the pass that begins, for an update that stands
+        before one.  Returns the stream and what is then pending for it, as a block does."""
+        raise NotImplementedError
+
+
 class Embedding(Part):
     """Token ids to the float32 residual stream."""
 
@@ -339,6 +363,7 @@ BLOCKS = Registry("block")
 EMBEDDINGS = Registry("embedding")
 HEADS = Registry("head")
 CONNECTIONS = Registry("connection")
+STREAM_UPDATES = Registry("stream update")
 Block.ROLE_REGISTRIES = {"mixer": MIXERS, "feed_forward": FEED_FORWARDS, "mixer_norm": NORMS,
                          "feed_forward_norm": NORMS}
 
@@ -350,6 +375,7 @@ register_block = BLOCKS.register
 register_embedding = EMBEDDINGS.register
 register_head = HEADS.register
 register_connection = CONNECTIONS.register
+register_stream_update = STREAM_UPDATES.register
 
 
 def build_part(registry: Registry, spec: PartSpec, *, hidden_size: int, dtype: torch.dtype,

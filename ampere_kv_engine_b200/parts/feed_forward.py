@@ -98,7 +98,7 @@ class GatedMLP(FeedForward):
 @register_feed_forward("dense_mlp")
 class DenseMLP(FeedForward):
     """``down(act(up(x)))`` without a gate.  params: ``intermediate_size``, ``activation`` (``"relu2"``: the square
-    of relu; ``"gelu_tanh"``; ``"silu"``), ``up`` / ``down`` (the matrices' names under the prefix, defaults
+    of relu; ``"gelu_tanh"``; ``"silu"``; ``"gelu"``), ``up`` / ``down`` (the matrices' names under the prefix, defaults
     ``up_proj.weight`` / ``down_proj.weight``)."""
 
     graph_safe = True
@@ -123,6 +123,28 @@ class DenseMLP(FeedForward):
     def load(self, tensors):
         self.up = tensors[self.up_name].contiguous()
         self.down = tensors[self.down_name].contiguous()
+
+    # A layer may run this part's two products together with those of a branch beside it.
+
+    def joinable(self) -> bool:
+        return True
+
+    def in_projection(self):
+        return self.up, None
+
+    def out_projection(self):
+        return self.down, None
+
+    def adopt(self, up, down):
+        """Views of larger matrices in place of the part's own."""
+        self.up, self.down = up, down
+
+    def heads_forward(self, x, ctx, projected=None, out=None):
+        """The activations before the second product.  ``projected``: (a product that holds the first one's columns, the
+        column where they begin); ``out``: (a wider matrix that receives the result, the first of its columns)."""
+        both, off = projected if projected is not None else (ops.linear(x, self.up, status=getattr(ctx, "status", None)), 0)
+        into = {} if out is None else {"out": out[0], "out_off": out[1]}
+        return ops.activation_columns(both, off, self.intermediate_size, self.activation, **into)
 
     def forward(self, x, ctx, residual=None):
         status = getattr(ctx, "status", None)

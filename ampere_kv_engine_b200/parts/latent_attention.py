@@ -4,11 +4,12 @@
     c_q = rmsnorm(a) * w_q;   c = rmsnorm(b) * w_kv;   r <- rotary(r)      (pairs of neighbouring dims)
     q   = W_uq c_q, per head [head_dim unrotated | rot_dim rotated];  the rotated part <- rotary(.)
     per head: k = W_uk c (unrotated) beside the shared r, v = W_uv c
-    s(i, j) = (q_unrot . k_j + q_rot . r_j) * scale,  i sees j iff 0 <= i - j (< window),  softmax
+    s(i, j) = (q_unrot . k_j + q_rot . r_j) * scale,  i sees j iff 0 <= i - j (< window),  softmax (with a sink: its
+              denominator also counts exp(sink_h))
     y       = W_o concat_h(sigmoid(g_h) sum_j p_j v_j)
 
 What of it a mixer has is up to its parameters: without ``q_rank`` the queries come straight from x (``W_q`` takes
-``W_dq``'s place in the first product); without ``gated`` there are no gates; without ``own_kv`` there is no ``W_dkv``
+``W_dq``'s place in the first product); without ``gated`` there are no gates, without ``sink`` no sinks; without ``own_kv`` there is no ``W_dkv``
 and the rows of an earlier schedule position (the model's schedule names it) are read, with this mixer's own queries,
 ``W_uk``, ``W_uv`` and window; the rotation may come with rescaled frequencies and a factor (``position_encoding``).
 
@@ -40,8 +41,8 @@ class LatentAttention(Mixer):
     and the width of the shared rotated key part), ``v_dim``, ``q_rank`` (None: queries straight from the input),
     ``kv_rank``, ``scale``, ``norm_eps``, ``rotary_base``, ``rotary_dims`` (how many of the ``rot_dim`` dims turn;
     default all) or ``position_encoding`` (a PartSpec of a rope in the pairs layout, in their place), ``window`` (None:
-    all keys), ``gated`` (bool: a sigmoid gate per head read from the input), ``own_kv`` (bool, default True), ``names``
-    (local tensor names)."""
+    all keys), ``gated`` (bool: a sigmoid gate per head read from the input), ``sink`` (bool: a learned number per head in
+    the softmax's denominator), ``own_kv`` (bool, default True), ``names`` (local tensor names)."""
 
     graph_safe = True
     takes_lazy_norm = True
@@ -49,7 +50,7 @@ class LatentAttention(Mixer):
 
     NAMES = {"dq": "q_a_proj.weight", "dq_norm": "q_a_norm.weight", "uq": "q_b_proj.weight", "q": "q_proj.weight",
              "dkv": "kv_a_proj.weight", "dkv_norm": "kv_a_norm.weight", "uk": "k_b_proj.weight",
-             "uv": "v_b_proj.weight", "gate": "gate_proj.weight", "out": "o_proj.weight"}
+             "uv": "v_b_proj.weight", "gate": "gate_proj.weight", "out": "o_proj.weight", "sink": "sinks"}
 
     def __init__(self, spec, **kw):
         super().__init__(spec, **kw)
@@ -83,6 +84,8 @@ class LatentAttention(Mixer):
         self.norm_eps = float(p.get("norm_eps", 1e-6))
         self.window = int(p["window"]) if p.get("window") else 0
         self.gated, self.own_kv = bool(p.get("gated", False)), bool(p.get("own_kv", True))
+        self.has_sink = bool(p.get("sink", False))
+        self.sink = None
         self.names = dict(self.NAMES, **(p.get("names") or {}))
         self.w_in = self.w_uq = self.w_uk = self.w_uv = self.w_o = self.q_norm = self.kv_norm = None
 
@@ -117,6 +120,8 @@ class LatentAttention(Mixer):
         specs[n["uv"]] = ParamSpec((H * self.v_dim, self.kv_rank))
         if self.gated:
             specs[n["gate"]] = ParamSpec((H, h))
+        if self.has_sink:
+            specs[n["sink"]] = ParamSpec((H,), kind="vector", init="around_zero")
         specs[n["out"]] = ParamSpec((h, H * self.v_dim))
         return specs
 
@@ -128,6 +133,8 @@ class LatentAttention(Mixer):
             self.kv_norm = tensors[n["dkv_norm"]]
         if self.gated:
             rows.append(tensors[n["gate"]])
+        if self.has_sink:
+            self.sink = tensors[n["sink"]].float().contiguous()
         spare = -sum(r.shape[0] for r in rows) % ROW_MULTIPLE
         if spare and not self.q_rank:
             rows.append(torch.zeros((spare, self.hidden_size), dtype=rows[0].dtype, device=rows[0].device))
@@ -166,7 +173,7 @@ class LatentAttention(Mixer):
                   out=q_row.view(tokens, H, self.row)[:, :, :rank].transpose(0, 1))
         mixed = torch.empty((tokens, H * rank), dtype=q.dtype, device=q.device)
         run_attention(ctx, group, q_row, rows, rows, mixed, num_heads=H, num_kv_heads=1, v_dim=rank, scale=self.scale,
-                      window=self.window, gate=gate)
+                      window=self.window, gate=gate, sink=self.sink)
         out = torch.empty((tokens, H * self.v_dim), dtype=q.dtype, device=q.device)
         torch.bmm(mixed.view(tokens, H, rank).transpose(0, 1), self.w_uv,
                   out=out.view(tokens, H, self.v_dim).transpose(0, 1))              # [H, tokens, v_dim]

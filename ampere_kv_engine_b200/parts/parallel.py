@@ -5,7 +5,8 @@ Each side is a registered mixer kind of its own.  The layer has one cache view, 
 side that keeps a state gets its share of the position's state (the sides' floats lie one behind the other in a
 request's slot).  When both sides offer ``heads_forward`` / ``out_projection`` (everything before the output
 projection, with an ``out_scale`` applied in float32 before the one rounding) and neither output projection has a
-bias, the two output projections run as one product over the sides' outputs laid next to each other; otherwise each
+bias, the two output projections run as one product over the sides' outputs laid next to each other (and likewise the
+first projections of sides that take theirs from a shared product); otherwise each
 side runs whole and ``ops.scaled_sum`` adds them up (sides with a bias on their output projection, or kinds that do
 not offer the two methods).
 
@@ -95,22 +96,76 @@ class ParallelMixers(Mixer):
         if self.out_norm is not None:
             self.norm_weights = tuple(tensors[self.out_norm[side]].float().contiguous() for side in ("left", "right"))
 
-    def _projected(self, x, ctx):
-        """One product for both sides' first projections, where both sides take theirs from a shared product and
-        neither has a bias there: ((product, first column of the left side's), (product, first column of the
-        right side's)), else (None, None)."""
+    def _shares_input(self) -> bool:
+        """Both sides take their first projections from a shared product, and neither has a bias there."""
+        return all(hasattr(m, "in_projection") and hasattr(m, "heads_forward") and hasattr(m, "out_projection")
+                   and (not hasattr(m, "joinable") or m.joinable() or self.out_norm is not None)
+                   and m.out_projection()[1] is None and m.in_projection()[1] is None for m in self.sides)
+
+    def _join_input(self):
+        """Both sides' first projections as one matrix, made once."""
         if self.w_in is None:
             self.w_in = False
-            if all(hasattr(m, "in_projection") and hasattr(m, "heads_forward") and hasattr(m, "out_projection")
-                   and m.out_projection()[1] is None and m.in_projection()[1] is None for m in self.sides):
+            if self._shares_input():
                 self.w_in = torch.cat([m.in_projection()[0] for m in self.sides], dim=0).contiguous()
                 self.in_split = self.sides[0].in_projection()[0].shape[0]
                 # the sides keep views of the one matrix, not copies of their parts
                 self.sides[0].w_in, self.sides[1].w_in = self.w_in[:self.in_split], self.w_in[self.in_split:]
-        if self.w_in is False:
+        return self.w_in
+
+    def _projected(self, x, ctx):
+        """One product for both sides' first projections, where both sides take theirs from a shared product and
+        neither has a bias there: ((product, first column of the left side's), (product, first column of the
+        right side's)), else (None, None)."""
+        if self._join_input() is False:
             return None, None
         both = ops.linear(x, self.w_in, status=ctx.status)
         return (both, 0), (both, self.in_split)
+
+    def _join_output(self):
+        """Both sides' output projections next to each other, made once."""
+        if self.w_o is None:
+            self.w_o = torch.cat([m.out_projection()[0] for m in self.sides], dim=1).contiguous()
+        return self.w_o
+
+    # A layer may run this part's first and last products together with those of a branch beside it.
+
+    def joinable(self) -> bool:
+        return self.joined and all(getattr(m, "joinable", None) is not None and m.joinable()
+                                   and getattr(m, "writes_into", False) for m in self.sides)
+
+    def in_projection(self):
+        return self._join_input(), None
+
+    def out_projection(self):
+        return self._join_output(), None
+
+    def adopt(self, w_in, w_o):
+        """Views of larger matrices in place of the part's own; the sides keep views of these."""
+        self.w_in, self.w_o = w_in, w_o
+        cols = self.sides[0].out_projection()[0].shape[1]
+        self.sides[0].adopt(w_in[:self.in_split], w_o[:, :cols])
+        self.sides[1].adopt(w_in[self.in_split:], w_o[:, cols:])
+
+    def heads_forward(self, x, ctx, cache, projected=None, out=None):
+        """Both sides' results before the output projection, side by side: [tokens, left columns + right columns].
+        ``projected`` and ``out`` as for the sides."""
+        cl, cr = self._views(cache)
+        left, right = self.sides
+        if projected is not None:
+            pl, pr = projected, (projected[0], projected[1] + self.in_split)
+        else:
+            pl, pr = self._projected(x, ctx)
+        shared = {} if pl is None else {"projected": pl}, {} if pr is None else {"projected": pr}
+        if not all(getattr(m, "writes_into", False) for m in self.sides):
+            return torch.cat((left.heads_forward(x, ctx, cl, **shared[0]), right.heads_forward(x, ctx, cr, **shared[1])), dim=1)
+        cols = left.out_projection()[0].shape[1]
+        if out is None:
+            out = (torch.empty((ctx.positions.shape[0], cols + right.out_projection()[0].shape[1]), dtype=self.dtype,
+                               device=self.device), 0)
+        left.heads_forward(x, ctx, cl, out=out, **shared[0])
+        right.heads_forward(x, ctx, cr, out=(out[0], out[1] + cols), **shared[1])
+        return out[0]
 
     @staticmethod
     def _float_output(side, x, ctx, cache, projected=None):
@@ -140,12 +195,10 @@ class ParallelMixers(Mixer):
                                        *self.norm_weights, eps=float(self.out_norm["eps"]), sa=self.scales[0],
                                        sb=self.scales[1], out_dtype=torch.float32)
         if self.joined:
-            if self.w_o is None:
-                self.w_o = torch.cat((left.out_projection()[0], right.out_projection()[0]), dim=1).contiguous()
-            both = torch.cat((left.heads_forward(x, ctx, cl), right.heads_forward(x, ctx, cr)), dim=1)
+            both, w_o = self.heads_forward(x, ctx, cache), self._join_output()
             if residual is not None:
-                summed = ops.linear_into_residual(both, self.w_o, residual, status=ctx.status)
+                summed = ops.linear_into_residual(both, w_o, residual, status=ctx.status)
                 if summed is not None:
                     return summed
-            return ops.linear(both, self.w_o, partial_ok=True, status=ctx.status)
+            return ops.linear(both, w_o, partial_ok=True, status=ctx.status)
         return ops.scaled_sum(left.forward(x, ctx, cl), right.forward(x, ctx, cr), *self.scales)

@@ -12,6 +12,11 @@ frequencies by wavelength (``scaling``): with ``turns(t) = rotary_dim * ln(origi
 ``ramp_j = clamp((j - lo) / max(hi - lo, 0.001), 0, 1)`` the frequency of pair j becomes
 ``f_j / factor * ramp_j + f_j * (1 - ramp_j)`` (slow pairs are stretched by ``factor``, fast ones kept) and cos and
 sin are multiplied by ``0.1 ln(factor) + 1``.  Such a table is formed in float64 and rounded once.
+
+A second rescaling by wavelength (``scaling`` with ``low`` and ``high``) has no factor on cos and sin: with the wavelength
+``l_j = 2 pi / f_j`` a frequency stays while ``l_j < original / high``, is divided by ``factor`` where
+``l_j > original / low``, and between the two is ``(1 - s) f_j / factor + s f_j`` with
+``s = (original / l_j - low) / (high - low)``; also formed in float64 and rounded once.
 """
 
 from __future__ import annotations
@@ -26,8 +31,9 @@ from .base import PositionEncoding, register_position_encoding
 @register_position_encoding("rope")
 class RotaryEmbedding(PositionEncoding):
     """params: ``theta``, ``rotary_dim``, ``layout`` (``"half"``, the default: dim i pairs with i + rotary_dim / 2;
-    ``"pairs"``: dim 2i with 2i + 1), ``scaling`` (None; ``factor`` alone: every frequency divided by it; or
-    ``factor``, ``original``, ``fast``, ``slow`` of the rescaling by wavelength)."""
+    ``"pairs"``: dim 2i with 2i + 1), ``scaling`` (None; ``factor`` alone: every frequency divided by it;
+    ``factor``, ``original``, ``fast``, ``slow`` of the first rescaling by wavelength; or ``factor``, ``original``,
+    ``low``, ``high`` of the second)."""
 
     graph_safe = True
 
@@ -56,6 +62,18 @@ class RotaryEmbedding(PositionEncoding):
         elif scaling is None:
             j = torch.arange(self.rotary_dim // 2, dtype=torch.float64)
             self.inv_freq = (self.theta ** (-2.0 * j / self.rotary_dim)).to(torch.float32).to(self.device)
+        elif "low" in scaling:
+            stretch, original = float(scaling["factor"]), float(scaling["original"])
+            low, high = float(scaling["low"]), float(scaling["high"])
+            if stretch <= 0 or original <= 0 or not 0 < low < high:
+                raise ValueError("rope: scaling needs a positive factor and original length and 0 < low < high")
+            j = torch.arange(self.rotary_dim // 2, dtype=torch.float64)
+            freq = self.theta ** (-2.0 * j / self.rotary_dim)
+            wave = 2.0 * math.pi / freq
+            mix = (original / wave - low) / (high - low)
+            between = (1.0 - mix) * freq / stretch + mix * freq
+            scaled = torch.where(wave > original / low, freq / stretch, torch.where(wave < original / high, freq, between))
+            self.inv_freq = scaled.to(torch.float32).to(self.device)
         else:
             stretch, original = float(scaling["factor"]), float(scaling["original"])
             if stretch <= 0 or original <= 0 or self.theta <= 1:

@@ -1,6 +1,6 @@
 """A feed-forward of many small gated experts of which every token uses a few, plus an optional shared expert.
 
-    z       = W_r x                         router logits, float32
+    z       = W_r x (+ bias)                router logits, float32
     s       = sigmoid(z)                    scores (``score="softmax"``: softmax of z over all experts)
     c       = s + correction                choice scores (the weights below use s)
     groups  : the experts form ``groups`` equal runs of neighbours; a group's score is the sum of its ``group_top``
@@ -10,7 +10,8 @@
     choices from ``experts`` on (``identity`` of them) are the identity: w_e x, no matrices; the router, the scores,
               the correction and the groups count them like experts
     expert  : g = min(W_gate x, limit); u = clamp(W_up x, -limit, limit); W_down (g * sigmoid(slope * g) * (u + 1))
-              (``activation="silu"``: plain W_down (silu(W_gate x) * W_up x), no clamp)
+              (``activation="silu"``: plain W_down (silu(W_gate x) * W_up x), no clamp; ``gated=False``:
+              W_down act(W_up x))
     y       = sum_e w_e expert_e(x)  +  shared(x)
 
 Everything runs on the device from the batch layout alone (no host read of the routing), so a decode step through it
@@ -35,16 +36,19 @@ class RoutedExperts(FeedForward):
     input, default 0), ``normalize`` (default True: the chosen scores are divided by their sum), ``route_scale``,
     ``weight_eps``, ``score`` (``"sigmoid"`` or
     ``"softmax"``), ``correction`` (bool, default True: a learned per-expert offset of the choice scores),
-    ``activation`` (``"clamped_swish"``, the default, with ``limit`` and ``swish_slope``; or ``"silu"``),
+    ``router_bias`` (bool, default False: a learned number per choice added to the logits), ``activation``
+    (``"clamped_swish"``, the default, with ``limit`` and ``swish_slope``; or ``"silu"``), ``gated`` (default True; False:
+    experts of one first matrix, ``activation`` then one of ``ops.ACTIVATIONS``, and no shared expert),
     ``intermediate_size`` of an expert, ``shared`` (None, or ``{"intermediate_size", "limit"}``), ``names`` (``expert`` with ``{}`` for
-    the index, ``gate``, ``up``, ``down``, ``router``, ``correction``, ``shared``)."""
+    the index, ``gate``, ``up``, ``down``, ``router``, ``router_bias``, ``correction``, ``shared``)."""
 
     graph_safe = True
     #: ``forward(..., defer_sum=True)`` hands back an ``ops.ExpertParts`` for a norm that adds the rows up itself
     defers_sum = True
 
     NAMES = {"expert": "experts.{}", "gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight",
-             "router": "router.weight", "correction": "router.correction", "shared": "shared_expert"}
+             "router": "router.weight", "router_bias": "router.bias", "correction": "router.correction",
+             "shared": "shared_expert"}
 
     def __init__(self, spec, **kw):
         super().__init__(spec, **kw)
@@ -69,7 +73,12 @@ class RoutedExperts(FeedForward):
         if self.score not in ops.MOE_SCORES:
             raise ValueError(f"routed_experts: score must be one of {sorted(ops.MOE_SCORES)}, got {self.score!r}")
         self.activation = str(p.get("activation", "clamped_swish"))
-        if self.activation not in ("clamped_swish", "silu"):
+        self.gated, self.has_router_bias = bool(p.get("gated", True)), bool(p.get("router_bias", False))
+        if not self.gated:
+            if self.activation not in ops.ACTIVATIONS or p.get("shared"):
+                raise ValueError(f"routed_experts: experts without a gate take an activation of {sorted(ops.ACTIVATIONS)} "
+                                 f"and no shared expert; got {self.activation!r}")
+        elif self.activation not in ("clamped_swish", "silu"):
             raise ValueError(f"routed_experts: activation must be 'clamped_swish' or 'silu', got {self.activation!r}")
         self.route_scale = float(p.get("route_scale", 1.0))
         self.weight_eps = float(p.get("weight_eps", 1e-20))
@@ -77,13 +86,16 @@ class RoutedExperts(FeedForward):
         self.intermediate_size = int(p["intermediate_size"])
         shared = p.get("shared")
         self.shared_size = int(shared["intermediate_size"]) if shared else 0
-        if self.activation == "silu":
+        if not self.gated:
+            self.limit = self.swish_slope = self.up_offset = self.shared_limit = 0.0
+        elif self.activation == "silu":
             # the clamped form with nothing to clamp, a slope of one and no offset on the up half is SiLU times up
             self.limit, self.swish_slope, self.up_offset, self.shared_limit = float("inf"), 1.0, 0.0, float("inf")
         else:
             self.limit, self.swish_slope, self.up_offset = float(p["limit"]), float(p.get("swish_slope", 1.702)), 1.0
             self.shared_limit = float(shared["limit"]) if shared else 0.0
         self.names = dict(self.NAMES, **(p.get("names") or {}))
+        self.router_bias = None
         self.w_router = self.correction = self.w_gate_up = self.w_down = self.shared_gate_up = self.shared_down = None
 
     def _expert(self, index: int, which: str) -> str:
@@ -93,10 +105,13 @@ class RoutedExperts(FeedForward):
         f, h, n = self.intermediate_size, self.hidden_size, self.names
         specs = {}
         for e in range(self.experts):
-            specs[self._expert(e, "gate")] = ParamSpec((f, h))
+            if self.gated:
+                specs[self._expert(e, "gate")] = ParamSpec((f, h))
             specs[self._expert(e, "up")] = ParamSpec((f, h))
             specs[self._expert(e, "down")] = ParamSpec((h, f))
         specs[n["router"]] = ParamSpec((self.choices, h))
+        if self.has_router_bias:
+            specs[n["router_bias"]] = ParamSpec((self.choices,), kind="vector", init="around_zero")
         if self.has_correction:
             specs[n["correction"]] = ParamSpec((self.choices,), kind="vector", init="around_zero")
         if self.shared_size:
@@ -109,7 +124,9 @@ class RoutedExperts(FeedForward):
         n = self.names
         # [experts, gate rows then up rows, hidden] and [experts, hidden, intermediate]
         self.w_gate_up = torch.stack([torch.cat((tensors[self._expert(e, "gate")], tensors[self._expert(e, "up")]), dim=0)
-                                      for e in range(self.experts)]).contiguous()
+                                      if self.gated else tensors[self._expert(e, "up")]
+                                      for e in range(self.experts)]).contiguous()      # (no gate rows: the up rows alone)
+        self.router_bias = tensors[n["router_bias"]].float().contiguous() if self.has_router_bias else None
         self.w_down = torch.stack([tensors[self._expert(e, "down")] for e in range(self.experts)]).contiguous()
         self.w_router = tensors[n["router"]].contiguous()
         self.correction = tensors[n["correction"]].float().contiguous() if self.has_correction else None
@@ -124,12 +141,15 @@ class RoutedExperts(FeedForward):
         chosen, weights = ops.moe_route(logits, self.correction, top=self.top, groups=self.groups,
                                         keep_groups=self.keep_groups, group_top=self.group_top,
                                         scale=self.route_scale, weight_eps=self.weight_eps, score=self.score,
-                                        normalize=self.normalize)
+                                        normalize=self.normalize, bias=self.router_bias)
         order, offsets = ops.moe_sort(chosen, self.choices)
         if self.identity:
             offsets = offsets[:self.experts + 1]       # the identity choices' pairs sort behind the experts' runs
-        act = ops.moe_gate_up(x, self.w_gate_up, order, offsets, top=self.top, limit=self.limit,
-                              slope=self.swish_slope, up_offset=self.up_offset)
+        if self.gated:
+            act = ops.moe_gate_up(x, self.w_gate_up, order, offsets, top=self.top, limit=self.limit,
+                                  slope=self.swish_slope, up_offset=self.up_offset)
+        else:
+            act = ops.moe_up(x, self.w_gate_up, order, offsets, top=self.top, activation=self.activation)
         parts = ops.moe_down(act, self.w_down, order, offsets, weights)
         shared = None
         if self.shared_size:

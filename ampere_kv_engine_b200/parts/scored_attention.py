@@ -162,7 +162,7 @@ class ScoredAttention(Mixer):
 
 def run_attention(ctx, group, q, k_cache, v_cache, out, *, num_heads, num_kv_heads, v_dim, scale, window=0, chunk=0,
                   softcap=0.0, slopes=None, gate=None, plain=False, keep_first=0, sigmoid_weights=False, head_bias=None,
-                  out_scale=1.0) -> None:
+                  out_scale=1.0, sink=None) -> None:
     """``ops.scored_attention`` over the step's tiles: the single-token tiles of a mixed step (they come first) apart
     from the prompt tiles, each with the number of key splits that fills the GPU.  ``plain``: nothing is done to the
     scores and the plain kernels take the sizes: ``ops.paged_attention`` runs instead."""
@@ -203,4 +203,4 @@ def run_attention(ctx, group, q, k_cache, v_cache, out, *, num_heads, num_kv_hea
             ctx.tile_nq[lo:hi], num_tiles=hi - lo, q_tile=q_tile, num_splits=splits, num_heads=num_heads,
             num_kv_heads=num_kv_heads, v_dim=v_dim, scale=scale, window=window, chunk=chunk, softcap=softcap,
             slopes=slopes, gate=gate, status=ctx.status, out=out, keep_first=keep_first,
-            sigmoid_weights=sigmoid_weights, head_bias=head_bias, out_scale=out_scale)
+            sigmoid_weights=sigmoid_weights, head_bias=head_bias, out_scale=out_scale, sink=sink)

@@ -17,7 +17,7 @@ import os
 import torch
 from safetensors import safe_open
 
-from ..parts.base import ParamSpec
+from ..parts.base import FREE_SIZE, ParamSpec
 
 _FLOAT_DTYPES = {"F32": torch.float32, "BF16": torch.bfloat16, "F16": torch.float16, "F64": torch.float64}
 _INT_DTYPES = {"I32": torch.int32, "I64": torch.int64, "I16": torch.int16, "I8": torch.int8, "U8": torch.uint8}
@@ -52,7 +52,7 @@ def check_against(specs: dict[str, ParamSpec], found: dict[str, tuple[tuple[int,
     missing = sorted(n for n, s in specs.items() if not s.optional and n not in found)
     unexpected = sorted(n for n in found if n not in specs)
     wrong_shape = sorted((n, specs[n].shape, found[n][0]) for n in found
-                         if n in specs and tuple(found[n][0]) != tuple(specs[n].shape))
+                         if n in specs and not specs[n].accepts(tuple(found[n][0])))
     wrong_dtype = []
     for n, (shape, dtype) in found.items():
         if n not in specs:
@@ -69,7 +69,8 @@ def check_against(specs: dict[str, ParamSpec], found: dict[str, tuple[tuple[int,
         lines.append(f"  unexpected ({len(unexpected)}): " + ", ".join(unexpected))
     if wrong_shape:
         lines.append(f"  wrong shape ({len(wrong_shape)}): " + ", ".join(
-            f"{n} is {list(got)}, expected {list(exp)}" for n, exp, got in wrong_shape))
+            f"{n} is {list(got)}, expected [{', '.join('any' if e == FREE_SIZE else str(e) for e in exp)}]"
+            for n, exp, got in wrong_shape))
     if wrong_dtype:
         lines.append(f"  wrong dtype ({len(wrong_dtype)}): " + ", ".join(f"{n} is {d}" for n, d in sorted(wrong_dtype)))
     raise WeightError("\n".join(lines))

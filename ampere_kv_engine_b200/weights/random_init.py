@@ -21,14 +21,14 @@ from .loader import cast_for
 
 def _draw(spec: ParamSpec, generator: torch.Generator, device) -> torch.Tensor:
     if spec.kind == "table":
-        return torch.zeros(spec.shape, dtype=torch.int32, device=device)
-    noise = torch.randn(spec.shape, generator=generator, dtype=torch.float32, device=device)
+        return torch.zeros(spec.drawn_shape(), dtype=torch.int32, device=device)
+    noise = torch.randn(spec.drawn_shape(), generator=generator, dtype=torch.float32, device=device)
     if spec.init == "norm":
         return 1.0 + 0.1 * noise
     if spec.init == "around_zero":
         return 0.1 * noise
     if spec.init == "unit_interval":
-        return torch.rand(spec.shape, generator=generator, dtype=torch.float32, device=device)
+        return torch.rand(spec.drawn_shape(), generator=generator, dtype=torch.float32, device=device)
     if spec.init == "zeros":
         return torch.zeros_like(noise)
     return 0.02 * noise

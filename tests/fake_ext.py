@@ -187,7 +187,7 @@ class FakeExt:
     def scored_attention(self, q, k_cache, v_cache, out, block_table, cu_q, ctx_lens, tile_seq, tile_q0, tile_nq,
                          partials, num_tiles, q_tile, num_splits, num_heads, num_kv_heads, v_dim, window, chunk, scale,
                          softcap, slopes=None, gate=None, status=None, kernel=0, keep_first=0, sigmoid_weights=False,
-                         head_bias=None, out_scale=1.0):
+                         head_bias=None, out_scale=1.0, sink=None):
         page_size = k_cache.shape[2]
         d = q.shape[1] // num_heads
         group = num_heads // num_kv_heads
@@ -228,7 +228,10 @@ class FakeExt:
                     scores = scores + head_bias.float()[:, None, None]
                 weights = torch.sigmoid(scores) * visible[None]
             else:
-                weights = torch.softmax(scores.masked_fill(~visible[None], -math.inf), -1)
+                scores = scores.masked_fill(~visible[None], -math.inf)
+                if sink is not None:      # one more score that belongs to no key
+                    scores = torch.cat((scores, sink.float()[:, None, None].expand(-1, n, 1)), dim=-1)
+                weights = torch.softmax(scores, -1)[..., :keys.numel()]
             o = torch.einsum("hts,shd->thd", weights, v.repeat_interleave(group, dim=1))
             if gate is not None:
                 o = o * gate[q0:q1].float()[:, :, None]
@@ -327,6 +330,8 @@ class FakeExt:
             y = torch.relu(z).square()
         elif kind == 1:
             y = 0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))
+        elif kind == 3:
+            y = 0.5 * z * (1 + torch.erf(z / math.sqrt(2)))
         else:
             y = z / (1 + torch.exp(-z))
         out.copy_(y.to(out.dtype))
@@ -334,7 +339,7 @@ class FakeExt:
     # ------------------------------------------------------------------ the gated delta rule
 
     def delta_prep(self, x, conv, rate_log, step_bias, state, cu_q, state_slots, qkv, coef, num_heads, num_kv_heads,
-                   head_dim, v_dim, taps, unit_eps):
+                   head_dim, v_dim, taps, unit_eps, steps=None, step_off=0, channel_decay=False, x_off=0, beta_off=None):
         from ampere_kv_engine_b200.kernels import ops
         G, D, H, V = num_kv_heads, head_dim, num_heads, v_dim
         channels = 2 * G * D + H * V
@@ -348,7 +353,7 @@ class FakeExt:
             if slot < 0 or q1 <= q0:
                 continue
             before = state[slot, memory:memory + (taps - 1) * channels].view(taps - 1, channels)
-            stream = torch.cat((before, xf[q0:q1, :channels]), dim=0)
+            stream = torch.cat((before, xf[q0:q1, x_off:x_off + channels]), dim=0)
             y = torch.zeros(q1 - q0, channels)
             for j in range(taps):
                 y = y + stream[j:j + q1 - q0] * conv[:, j]
@@ -357,18 +362,26 @@ class FakeExt:
             q = q * torch.rsqrt(q.square().sum(-1, keepdim=True) + unit_eps) * D ** -0.5
             k = k * torch.rsqrt(k.square().sum(-1, keepdim=True) + unit_eps)
             qkv[q0:q1] = torch.cat((q.reshape(q1 - q0, -1), k.reshape(q1 - q0, -1), y[:, 2 * G * D:]), dim=1)
-            tail = xf[q0:q1, channels + H * V:]
-            coef[q0:q1, :H] = torch.sigmoid(tail[:, :H])
-            coef[q0:q1, H:] = torch.exp(-torch.exp(rate_log) * torch.nn.functional.softplus(tail[:, H:] + step_bias))
+            count = H * D if channel_decay else H
+            if steps is None:
+                step, beta = xf[q0:q1, channels + H * V + H:], xf[q0:q1, channels + H * V:channels + H * V + H]
+            else:
+                step, beta = steps[q0:q1, step_off:step_off + count].float(), xf[q0:q1, beta_off:beta_off + H]
+            rate = torch.exp(rate_log).repeat_interleave(count // H)
+            coef[q0:q1, :H] = torch.sigmoid(beta)
+            coef[q0:q1, H:] = torch.exp(-rate * torch.nn.functional.softplus(step + step_bias))
 
     def delta_scan(self, qkv, coef, x, norm_weight, state, cu_q, state_slots, scratch, out, num_heads, num_kv_heads,
-                   head_dim, v_dim, taps, norm_eps):
+                   head_dim, v_dim, taps, norm_eps, gates=None, gate_off=0, gate_kind=0, channel_decay=False, x_off=0,
+                   out_off=0, factor=1.0):
         from ampere_kv_engine_b200.kernels import ops
         G, D, H, V = num_kv_heads, head_dim, num_heads, v_dim
         channels = 2 * G * D + H * V
         memory = ops.delta_state_floats(H, G, D, V, taps)[0]      # the stand-in keeps S in the first H * D * V floats of it
         cu, slots = cu_q.tolist(), state_slots.tolist()
-        out.zero_()
+        out[:, out_off:out_off + H * V] = 0
+        if gates is None:
+            gates, gate_off = x, channels
         for s, slot in enumerate(slots):
             q0, q1 = cu[s], cu[s + 1]
             if slot < 0 or q1 <= q0:
@@ -377,19 +390,20 @@ class FakeExt:
             for t in range(q0, q1):
                 q, k = qkv[t, :G * D].view(G, D), qkv[t, G * D:2 * G * D].view(G, D)
                 v = qkv[t, 2 * G * D:].view(H, V)
-                gate = x[t, channels:channels + H * V].float().view(H, V)
+                gate = gates[t, gate_off:gate_off + H * V].float().view(H, V)
+                gate = torch.sigmoid(gate) * (gate if gate_kind == 0 else 1.0) * factor
                 for h in range(H):
                     j = h // (H // G)
-                    S[h] = S[h] * coef[t, H + h]
+                    S[h] = S[h] * (coef[t, H + h * D:H + (h + 1) * D, None] if channel_decay else coef[t, H + h])
                     u = coef[t, h] * (v[h] - S[h].T @ k[j])
                     S[h] = S[h] + torch.outer(k[j], u)
                     o = S[h].T @ q[j]
-                    o = o * torch.rsqrt(o.square().mean() + norm_eps) * norm_weight * (gate[h] * torch.sigmoid(gate[h]))
-                    out[t, h * V:(h + 1) * V] = o.to(out.dtype)
+                    o = o * torch.rsqrt(o.square().mean() + norm_eps) * norm_weight * gate[h]
+                    out[t, out_off + h * V:out_off + (h + 1) * V] = o.to(out.dtype)
             state[slot, :H * D * V] = S.reshape(-1)
             if taps > 1:
                 before = state[slot, memory:memory + (taps - 1) * channels].view(taps - 1, channels)
-                stream = torch.cat((before, x[q0:q1, :channels].float()), dim=0)
+                stream = torch.cat((before, x[q0:q1, x_off:x_off + channels].float()), dim=0)
                 state[slot, memory:memory + (taps - 1) * channels] = stream[-(taps - 1):].reshape(-1)
 
     # ------------------------------------------------------------------ rotary positions, linear memories, the stream
@@ -543,15 +557,85 @@ class FakeExt:
             out[q0:q1, 2 * gn + inner:2 * gn + inner + H] = torch.exp(-torch.exp(rate_log) * dt)
             out[q0:q1, 2 * gn + inner + H:2 * gn + 2 * inner + H] = y[:, :inner]
 
-    def conv_tail(self, x, state, tail_off, cu_q, state_slots, conv_off, channels, taps):
+    def conv_tail(self, x, state, tail_off, cu_q, state_slots, conv_off, channels, taps, bias=None):
         cu, slots = cu_q.tolist(), state_slots.tolist()
         for s, slot in enumerate(slots):
             q0, q1 = cu[s], cu[s + 1]
             if slot < 0 or q1 <= q0:
                 continue
             before = state[slot, tail_off:tail_off + (taps - 1) * channels].view(taps - 1, channels)
-            stream = torch.cat((before, x[q0:q1, conv_off:conv_off + channels].float()), dim=0)
+            rows = x[q0:q1, conv_off:conv_off + channels].float()
+            stream = torch.cat((before, rows if bias is None else rows + bias), dim=0)
             state[slot, tail_off:tail_off + (taps - 1) * channels] = stream[stream.shape[0] - (taps - 1):].reshape(-1)
+
+    def conv_rotary_prep(self, x, x_off, bias, conv, state, tail_off, cu_q, state_slots, positions, slots, freq, q_out,
+                         k_cache, v_cache, num_heads, num_kv_heads, head_dim, v_dim, taps, rotary_dims, layout, factor,
+                         keep_tail, status=None):
+        NH, G, D, V = num_heads, num_kv_heads, head_dim, v_dim
+        channels = (NH + G) * D + G * V
+        u = x[:, x_off:x_off + channels].float()
+        u = u if bias is None else u + bias
+        y = torch.zeros_like(u)
+        cu, held = cu_q.tolist(), state_slots.tolist()
+        for s, slot in enumerate(held):
+            q0, q1 = cu[s], cu[s + 1]
+            before = torch.zeros(taps - 1, channels)
+            if slot >= 0 and taps > 1:
+                before = state[slot, tail_off:tail_off + (taps - 1) * channels].view(taps - 1, channels).clone()
+            stream = torch.cat((before, u[q0:q1]), dim=0)
+            for j in range(taps):
+                y[q0:q1] += stream[j:j + q1 - q0] * conv[:, j]
+            if keep_tail and slot >= 0 and taps > 1:
+                state[slot, tail_off:tail_off + (taps - 1) * channels] = stream[-(taps - 1):].reshape(-1)
+        half = rotary_dims // 2
+        angle = positions.float()[:, None] * freq[None, :]
+        cos, sin = (angle.cos() * factor)[:, None, :], (angle.sin() * factor)[:, None, :]
+
+        def turn(t):
+            t = t.clone()
+            a, b = (slice(0, half), slice(half, rotary_dims)) if layout == 0 else (slice(0, rotary_dims, 2), slice(1, rotary_dims, 2))
+            p, q = t[..., a].clone(), t[..., b].clone()
+            t[..., a], t[..., b] = p * cos - q * sin, q * cos + p * sin
+            return t
+
+        n = x.shape[0]
+        q_out.copy_(turn(y[:, :NH * D].view(n, NH, D)).reshape(n, -1).to(q_out.dtype))
+        k, v = turn(y[:, NH * D:(NH + G) * D].view(n, G, D)), y[:, (NH + G) * D:].view(n, G, V)
+        self._write(k.to(k_cache.dtype), v.to(v_cache.dtype), slots, k_cache, v_cache)
+
+    def gate_columns(self, values, x, gate_off, out, out_off, factor=1.0):
+        w = values.shape[1]
+        g = torch.sigmoid(x[:, gate_off:gate_off + w].float())
+        out[:, out_off:out_off + w] = (values.float() * g * factor).to(out.dtype)
+
+    def activation_columns(self, x, off, width, kind, out, out_off):
+        y = torch.empty(x.shape[0], width, dtype=x.dtype)
+        self.activation(x[:, off:off + width], y, kind)
+        out[:, out_off:out_off + width] = y
+
+    def stream_sum(self, hidden, a, b, parts, shared, top, copy):
+        for t in (a, b):
+            if t is not None:
+                hidden += t.float()
+        if parts is not None:
+            rows = parts.view(-1, top, parts.shape[1]).sum(1)
+            hidden += rows if shared is None else rows + shared.float()
+        if copy is not None:
+            copy.copy_(hidden.to(copy.dtype))
+
+    def stream_concat(self, hidden, start, out):
+        out.copy_(torch.cat((hidden, start), dim=1).to(out.dtype))
+
+    def stream_row_add(self, hidden, row):
+        hidden += row
+
+    def token_gate(self, z, ids, sampled, table, col_off, out, status=None):
+        ids = ids.long()
+        if sampled is not None:
+            ids = torch.where(ids < 0, sampled.long()[(-ids - 1).clamp(min=0)], ids)
+        g = z.float()
+        g = 0.5 * g * (1 + torch.tanh(math.sqrt(2 / math.pi) * (g + 0.044715 * g ** 3)))
+        out.copy_((g * table[ids][:, col_off:col_off + z.shape[1]].float()).to(out.dtype))
 
     @staticmethod
     def _hyper_write(x, y, mix, write, scale):
@@ -606,8 +690,10 @@ class FakeExt:
     # ------------------------------------------------------------------ routed experts
 
     def moe_route(self, logits, correction, chosen, weights, groups, keep_groups, group_top, scale, weight_eps,
-                  score_kind=0, normalize=True):
+                  score_kind=0, normalize=True, bias=None):
         n, E = logits.shape
+        if bias is not None:
+            logits = logits + bias
         top = chosen.shape[1]
         s = torch.sigmoid(logits.float()) if score_kind == 0 else torch.softmax(logits.float(), dim=-1)
         c = s if correction is None else s + correction
@@ -644,6 +730,16 @@ class FakeExt:
             both = x[rows // top].float() @ w_gate_up[e].float().T
             g, u = both[:, :inter].clamp(max=limit), both[:, inter:].clamp(min=-limit, max=limit)
             act[off[e]:off[e + 1]] = (g * torch.sigmoid(slope * g) * (u + up_offset)).to(act.dtype)
+
+    def moe_up(self, x, w_up, order, offsets, act, top, activation, form=0):
+        off = offsets.tolist()
+        for e in range(len(off) - 1):
+            rows = order[off[e]:off[e + 1]].long()
+            if rows.numel():
+                z = x[rows // top].float() @ w_up[e].float().T
+                y = torch.empty_like(z)
+                self.activation(z, y, activation)
+                act[off[e]:off[e + 1]] = y.to(act.dtype)
 
     def moe_down(self, act, w_down, order, offsets, weights, out, form=0):
         off = offsets.tolist()
