@@ -10,6 +10,8 @@ failed step reserved are given back; the reference offers no such rollback
 
 from __future__ import annotations
 
+import gc
+
 import torch
 
 from ..cache.manager import CacheManager, SequenceCache
@@ -192,8 +194,16 @@ class ModelRunner:
         torch.cuda.synchronize(self.device)
         graph = torch.cuda.CUDAGraph()
         before = ops.launch_count
-        with torch.cuda.graph(graph, pool=self._graph_pool):
-            logits = self.model.forward(ctx, self.views)
+        # an older engine's graphs must not be released by the garbage collector in the middle of a capture: the
+        # driver refuses that and the capture is lost
+        collecting = gc.isenabled()
+        gc.disable()
+        try:
+            with torch.cuda.graph(graph, pool=self._graph_pool):
+                logits = self.model.forward(ctx, self.views)
+        finally:
+            if collecting:
+                gc.enable()
         launches = ops.launch_count - before
         graph.replay()
         captured = _CapturedDecode(layout, dev, ctx, graph, logits, launches)

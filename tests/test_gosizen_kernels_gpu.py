@@ -470,13 +470,15 @@ def test_the_mixture_as_a_layer_uses_it(dtype, tokens, width, ff, experts, top):
         status = None
     want = plain.experts_mixture(x.double(), w, "mlp", mlp)
     got = part.forward(x.cuda().to(dtype), Ctx())
-    torch.testing.assert_close(got.double().cpu(), want, **TOL[dtype])
+    # up to four experts' activations, each rounded once, in a sum of unit size
+    tol = TOL[dtype] if dtype == torch.float32 else dict(atol=4e-2, rtol=2e-2)
+    torch.testing.assert_close(got.double().cpu(), want, **tol)
     # summed into the stream by the kernel that adds up a layer's branches
     hidden = torch.randn((x.shape[0], width), generator=g)
     other = torch.randn((x.shape[0], width), generator=g).to(dtype)
     stream = hidden.cuda()
     copy = _ops().stream_sum(stream, [other.cuda(), part.forward(x.cuda().to(dtype), Ctx(), defer_sum=True)], copy_dtype=dtype)
-    torch.testing.assert_close(stream.double().cpu(), hidden.double() + other.double() + want, **TOL[dtype])
+    torch.testing.assert_close(stream.double().cpu(), hidden.double() + other.double() + want, **tol)
     torch.testing.assert_close(copy, stream.to(dtype), atol=0, rtol=0)
 
 
