@@ -10,7 +10,8 @@
 //
 // A block takes a run of up to kRun tokens and some of their heads, a warp a head at a time: a lane holds the taps of a
 // pair of channels in registers and walks the run's tokens with the last taps - 1 inputs beside them, so that every
-// input is read once; cos and sin of the run's positions are worked out once per block.  Where every sequence of the
+// input is read once; cos and sin of the run's positions are worked out once per block.  (Prompts, where pairs of channels
+// start on boundaries of their size: two neighbouring channels per access, all inputs of a run loaded ahead.)  Where every sequence of the
 // step has one token (decoding) a thread also stores its channel's last taps - 1 inputs into the state slot; otherwise
 // conv_tail does that afterwards.
 //
@@ -92,17 +93,11 @@ __device__ __forceinline__ float channel_step(const ConvPrepParams& p, Channel<T
   return y;
 }
 
-template <typename T, int TAPS>
-__global__ void __launch_bounds__(kConvWarps * 32) conv_rotary_prep_kernel(ConvPrepParams p) {
-  extern __shared__ __align__(16) float2 turn[];             // [kRun][half]: cos and sin (times the factor)
-  __shared__ TokenInfo infos[kRun];
-  __shared__ int64_t cache_rows[kRun];                       // page and offset of the token, or -1
-  pdl_launch_dependents();
-  pdl_wait();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int NH = p.num_heads, NKV = p.num_kv_heads, D = p.head_dim, DV = p.v_dim, half = p.rotary_dims / 2;
-  const int64_t token0 = (int64_t)blockIdx.x * p.run;
-  const int run = (int)(p.num_tokens - token0 < p.run ? p.num_tokens - token0 : p.run);
+// What a block knows of its run of tokens: where each stands in its sequence, the cache row of each token's first kv head
+// (or -1: not stored), and cos and sin of its positions.
+__device__ __forceinline__ void run_prologue(const ConvPrepParams& p, int64_t token0, int run, TokenInfo* infos,
+                                             int64_t* cache_rows, float2* turn) {
+  const int half = p.rotary_dims / 2;
   if (threadIdx.x < run) {
     const int64_t token = token0 + threadIdx.x;
     int lo = 0, hi = p.num_seqs;                             // cu_q[lo] <= token < cu_q[hi]
@@ -117,12 +112,14 @@ __global__ void __launch_bounds__(kConvWarps * 32) conv_rotary_prep_kernel(ConvP
     info.slot = slot < p.num_slots ? slot : -1;
     info.fresh = threadIdx.x == 0 || info.offset == 0;
     infos[threadIdx.x] = info;
-    const int64_t at = p.slots != nullptr ? p.slots[token] : -1;
-    cache_rows[threadIdx.x] = at;
-    if (at >= 0 && at / p.page_size >= p.num_pages) {
-      set_status(p.status, kBadSlot);
-      cache_rows[threadIdx.x] = -1;
+    const int at = p.slots != nullptr ? p.slots[token] : -1;
+    int64_t row = -1;
+    if (at >= 0) {
+      const int page = at / p.page_size;
+      if (page >= p.num_pages) set_status(p.status, kBadSlot);
+      else row = (int64_t)page * p.num_kv_heads * p.page_size + at % p.page_size;
     }
+    cache_rows[threadIdx.x] = row;
   }
   for (int i = threadIdx.x; i < run * half; i += blockDim.x) {
     const int t = i / half, pair = i - t * half;
@@ -131,6 +128,20 @@ __global__ void __launch_bounds__(kConvWarps * 32) conv_rotary_prep_kernel(ConvP
     turn[i] = make_float2(c * p.factor, s * p.factor);
   }
   __syncthreads();
+}
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(kConvWarps * 32) conv_rotary_prep_kernel(ConvPrepParams p) {
+  extern __shared__ __align__(16) float2 turn[];             // [kRun][half]: cos and sin (times the factor)
+  __shared__ TokenInfo infos[kRun];
+  __shared__ int64_t cache_rows[kRun];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int NH = p.num_heads, NKV = p.num_kv_heads, D = p.head_dim, DV = p.v_dim, half = p.rotary_dims / 2;
+  const int64_t token0 = (int64_t)blockIdx.x * p.run;
+  const int run = (int)(p.num_tokens - token0 < p.run ? p.num_tokens - token0 : p.run);
+  run_prologue(p, token0, run, infos, cache_rows, turn);
   for (int h = blockIdx.y * kConvWarps + warp; h < NH + 2 * NKV; h += gridDim.y * kConvWarps) {
     const bool is_q = h < NH, is_v = h >= NH + NKV;
     const int g = is_q ? h : (is_v ? h - NH - NKV : h - NH);
@@ -138,9 +149,8 @@ __global__ void __launch_bounds__(kConvWarps * 32) conv_rotary_prep_kernel(ConvP
     const int first = is_q ? g * D : (is_v ? (NH + NKV) * D + g * DV : NH * D + g * D);
     auto row_of = [&](int t) -> T* {
       if (is_q) return (T*)p.q_out + ((token0 + t) * NH + g) * (int64_t)D;
-      const int64_t at = cache_rows[t];
-      if (at < 0) return nullptr;
-      const int64_t row = (at / p.page_size * NKV + g) * p.page_size + at % p.page_size;
+      if (cache_rows[t] < 0) return nullptr;
+      const int64_t row = cache_rows[t] + (int64_t)g * p.page_size;
       return is_v ? (T*)p.v_cache + row * p.v_row_stride : (T*)p.k_cache + row * p.k_row_stride;
     };
     const int turned = is_v ? 0 : half;
@@ -172,6 +182,160 @@ __global__ void __launch_bounds__(kConvWarps * 32) conv_rotary_prep_kernel(ConvP
   }
 }
 
+// Two neighbouring elements in one access
+template <typename T>
+__device__ __forceinline__ float2 load2(const T* p);
+template <>
+__device__ __forceinline__ float2 load2<float>(const float* p) { return *reinterpret_cast<const float2*>(p); }
+template <>
+__device__ __forceinline__ float2 load2<__nv_bfloat16>(const __nv_bfloat16* p) {
+  const uint32_t raw = *reinterpret_cast<const uint32_t*>(p);
+  return make_float2(__uint_as_float(raw << 16), __uint_as_float(raw & 0xffff0000u));
+}
+template <typename T>
+__device__ __forceinline__ void store2(T* p, float a, float b);
+template <>
+__device__ __forceinline__ void store2<float>(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+template <>
+__device__ __forceinline__ void store2<__nv_bfloat16>(__nv_bfloat16* p, float a, float b) {
+  const __nv_bfloat162 pair = __floats2bfloat162_rn(a, b);
+  *reinterpret_cast<uint32_t*>(p) = *reinterpret_cast<const uint32_t*>(&pair);
+}
+
+// The prompts' form: a run of kRun tokens of one sequence.  A lane takes two neighbouring channels (and the two that
+// they turn with): all inputs of the run, and the taps - 1 before it, are on their way before the first is used.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(kConvWarps * 32) conv_rotary_prep_run_kernel(ConvPrepParams p) {
+  extern __shared__ __align__(16) float2 turn[];
+  __shared__ TokenInfo infos[kRun];
+  __shared__ int64_t cache_rows[kRun];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int NH = p.num_heads, NKV = p.num_kv_heads, D = p.head_dim, DV = p.v_dim, half = p.rotary_dims / 2;
+  const int64_t token0 = (int64_t)blockIdx.x * kRun;
+  const int run = (int)(p.num_tokens - token0 < kRun ? p.num_tokens - token0 : kRun);
+  run_prologue(p, token0, run, infos, cache_rows, turn);
+  constexpr int kKeep = TAPS - 1;
+  // the channel pair c of the run: u[0 .. kKeep) before the run, then the run's own
+  auto inputs = [&](int c, float2 (&u)[kKeep + kRun]) {
+    const T* x = (const T*)p.x + c;
+    float2 bias = make_float2(0.f, 0.f);
+    if (p.bias != nullptr) bias = *reinterpret_cast<const float2*>(p.bias + c);
+#pragma unroll
+    for (int t = 0; t < kRun; ++t) {
+      u[kKeep + t] = make_float2(0.f, 0.f);
+      if (t < run) u[kKeep + t] = load2<T>(x + (token0 + t) * p.x_stride);
+    }
+    const TokenInfo info = infos[0];
+#pragma unroll
+    for (int j = 0; j < kKeep; ++j) {
+      const int back = info.offset - kKeep + j;
+      u[j] = make_float2(0.f, 0.f);
+      if (back >= 0) {
+        u[j] = load2<T>(x + (info.first + back) * p.x_stride);
+        u[j].x += bias.x;
+        u[j].y += bias.y;
+      } else if (info.slot >= 0) {
+        const float* before = p.state + (int64_t)info.slot * p.state_stride + p.tail_off + (int64_t)(kKeep + back) * p.channels + c;
+        u[j] = make_float2(before[0], before[1]);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < kRun; ++t) {
+      u[kKeep + t].x += bias.x;
+      u[kKeep + t].y += bias.y;
+    }
+  };
+  auto taps_of = [&](int c, float2 (&w)[TAPS]) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = make_float2(p.conv[(int64_t)c * TAPS + j], p.conv[(int64_t)(c + 1) * TAPS + j]);
+  };
+  // the inputs that the convolution of the run's token t sees: a token that is its sequence's first (or one of the
+  // first few) has zeros, or what its own slot holds, in place of another sequence's inputs
+  auto convolve = [&](const float2 (&u)[kKeep + kRun], const float2 (&w)[TAPS], int t, int c) -> float2 {
+    float2 y = make_float2(0.f, 0.f);
+    const TokenInfo info = infos[t];
+    const int own = info.offset < t ? info.offset : t;          // inputs of this sequence inside the run before t
+    if (own == t || own >= kKeep) {
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        y.x = fmaf(w[j].x, u[t + j].x, y.x);
+        y.y = fmaf(w[j].y, u[t + j].y, y.y);
+      }
+      return y;
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      const int back = info.offset - kKeep + j;
+      float2 v = make_float2(0.f, 0.f);
+      if (back >= 0) {
+        v = u[t + j];
+      } else if (info.slot >= 0) {
+        const float* before = p.state + (int64_t)info.slot * p.state_stride + p.tail_off + (int64_t)(kKeep + back) * p.channels + c;
+        v = make_float2(before[0], before[1]);
+      }
+      y.x = fmaf(w[j].x, v.x, y.x);
+      y.y = fmaf(w[j].y, v.y, y.y);
+    }
+    return y;
+  };
+  for (int h = blockIdx.y * kConvWarps + warp; h < NH + 2 * NKV; h += gridDim.y * kConvWarps) {
+    const bool is_q = h < NH, is_v = h >= NH + NKV;
+    const int g = is_q ? h : (is_v ? h - NH - NKV : h - NH);
+    const int width = is_v ? DV : D;
+    const int first = is_q ? g * D : (is_v ? (NH + NKV) * D + g * DV : NH * D + g * D);
+    auto row_of = [&](int t) -> T* {
+      if (is_q) return (T*)p.q_out + ((token0 + t) * NH + g) * (int64_t)D;
+      if (cache_rows[t] < 0) return nullptr;
+      const int64_t row = cache_rows[t] + (int64_t)g * p.page_size;
+      return is_v ? (T*)p.v_cache + row * p.v_row_stride : (T*)p.k_cache + row * p.k_row_stride;
+    };
+    const int turned = is_v ? 0 : half;
+    for (int i = 2 * lane; i < turned; i += 64) {
+      float2 ua[kKeep + kRun], ub[kKeep + kRun], wa[TAPS], wb[TAPS];
+      inputs(first + i, ua);
+      inputs(first + half + i, ub);
+      taps_of(first + i, wa);
+      taps_of(first + half + i, wb);
+#pragma unroll
+      for (int t = 0; t < kRun; ++t) {
+        if (t >= run) break;
+        const float2 a = convolve(ua, wa, t, first + i), b = convolve(ub, wb, t, first + half + i);
+        const float4 cs = *reinterpret_cast<const float4*>(turn + t * half + i);       // cos, sin of two pairs
+        T* dst = row_of(t);
+        if (dst != nullptr) {
+          store2<T>(dst + i, a.x * cs.x - b.x * cs.y, a.y * cs.z - b.y * cs.w);
+          store2<T>(dst + half + i, b.x * cs.x + a.x * cs.y, b.y * cs.z + a.y * cs.w);
+        }
+      }
+    }
+    for (int d = 2 * turned + 2 * lane; d < width; d += 64) {
+      float2 u[kKeep + kRun], w[TAPS];
+      inputs(first + d, u);
+      taps_of(first + d, w);
+#pragma unroll
+      for (int t = 0; t < kRun; ++t) {
+        if (t >= run) break;
+        const float2 y = convolve(u, w, t, first + d);
+        T* dst = row_of(t);
+        if (dst != nullptr) store2<T>(dst + d, y.x, y.y);
+      }
+    }
+  }
+}
+
+// whether every pair of channels the runs' form reads and writes at once starts on a boundary of its size
+template <typename T>
+bool conv_runs_take(const ConvPrepParams& p) {
+  auto even = [](int64_t v) { return v % 2 == 0; };
+  auto placed = [](const void* q, int bytes) { return reinterpret_cast<uintptr_t>(q) % bytes == 0; };
+  const int pair = 2 * (int)sizeof(T);
+  return p.layout == 0 && p.taps <= 4 && even(p.rotary_dims / 2) && even(p.head_dim) && even(p.v_dim) && even(p.x_stride) &&
+         even(p.k_row_stride) && even(p.v_row_stride) && placed(p.x, pair) && placed(p.q_out, pair) && placed(p.k_cache, pair) &&
+         placed(p.v_cache, pair) && placed(p.bias, 8);
+}
+
 template <typename T>
 int launch_conv_prep_typed(const ConvPrepParams& p, cudaStream_t stream) {
   ConvPrepParams q = p;
@@ -180,6 +344,17 @@ int launch_conv_prep_typed(const ConvPrepParams& p, cudaStream_t stream) {
   q.run = p.num_tokens < 256 || p.keep_tail ? 1 : kRun;
   int across = 1;
   const int64_t runs = (p.num_tokens + q.run - 1) / q.run;
+  if (q.run == kRun && conv_runs_take<T>(p)) {
+    const dim3 grid((unsigned)runs, (unsigned)((heads + 2 * kConvWarps - 1) / (2 * kConvWarps))), block(kConvWarps * 32);
+    const size_t smem = (size_t)kRun * (p.rotary_dims / 2) * sizeof(float2);
+    if (runs > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
+    switch (p.taps) {
+      case 1: return (int)launch_chain(conv_rotary_prep_run_kernel<T, 1>, grid, block, smem, stream, dim3(1, 1, 1), q);
+      case 2: return (int)launch_chain(conv_rotary_prep_run_kernel<T, 2>, grid, block, smem, stream, dim3(1, 1, 1), q);
+      case 3: return (int)launch_chain(conv_rotary_prep_run_kernel<T, 3>, grid, block, smem, stream, dim3(1, 1, 1), q);
+      default: return (int)launch_chain(conv_rotary_prep_run_kernel<T, 4>, grid, block, smem, stream, dim3(1, 1, 1), q);
+    }
+  }
   while (across < 16 && runs * across < 512 && heads > across * kConvWarps) across *= 2;
   if (runs > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
   const dim3 grid((unsigned)runs, (unsigned)across), block(kConvWarps * 32);

@@ -643,17 +643,21 @@ __global__ void __launch_bounds__(kGemvWarps * 32) moe_gemv_kernel(MoeGemmParams
       const int64_t src = FIRST ? (int64_t)(pair[r] / p.top) : (int64_t)sorted;
       x[r] = reinterpret_cast<const uint4*>(a + src * K);
     }
-    for (int f = 0; f < kPerWarp; ++f) {
+    // two weight rows at a time: a feature's gate and up row, or two features
+    constexpr int kRowsAtOnce = 2, kStep = GATED ? 1 : 2;
+    for (int f = 0; f < kPerWarp; f += kStep) {
       const int feature = blockIdx.x * kGemvFeatures + warp * kPerWarp + f;
       if (feature >= N) break;                                    // the same for the whole warp
-      const uint4* wg = reinterpret_cast<const uint4*>(w + (int64_t)feature * K);
-      const uint4* wu = GATED ? reinterpret_cast<const uint4*>(w + (int64_t)(N + feature) * K) : wg;
-      float acc[GATED ? 2 : 1][kGemvRows] = {};
+      const bool pairs = GATED || feature + 1 < N;
+      const uint4* wr[kRowsAtOnce];
+      wr[0] = reinterpret_cast<const uint4*>(w + (int64_t)feature * K);
+      wr[1] = reinterpret_cast<const uint4*>(w + (int64_t)(GATED ? N + feature : (pairs ? feature + 1 : feature)) * K);
+      float acc[kRowsAtOnce][kGemvRows] = {};
 #pragma unroll 2
       for (int c = lane; c < chunks; c += 32) {
         float g[8], u[8];
-        unpack8(wg[c], g);
-        if (GATED) unpack8(wu[c], u);
+        unpack8(wr[0][c], g);
+        unpack8(wr[1][c], u);
 #pragma unroll
         for (int r = 0; r < kGemvRows; ++r) {
           float v[8];
@@ -661,38 +665,39 @@ __global__ void __launch_bounds__(kGemvWarps * 32) moe_gemv_kernel(MoeGemmParams
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
             acc[0][r] = fmaf(g[i], v[i], acc[0][r]);
-            if (GATED) acc[GATED ? 1 : 0][r] = fmaf(u[i], v[i], acc[GATED ? 1 : 0][r]);
+            acc[1][r] = fmaf(u[i], v[i], acc[1][r]);
           }
         }
       }
 #pragma unroll
       for (int r = 0; r < kGemvRows; ++r) {
         acc[0][r] = warp_sum(acc[0][r]);
-        if (GATED) acc[GATED ? 1 : 0][r] = warp_sum(acc[GATED ? 1 : 0][r]);
+        acc[1][r] = warp_sum(acc[1][r]);
       }
       if (lane < count) {
         float first = 0.f, second = 0.f;
+        int mine = pair[0];
 #pragma unroll
         for (int r = 0; r < kGemvRows; ++r) {
           if (r == lane) {
             first = acc[0][r];
-            second = acc[GATED ? 1 : 0][r];
+            second = acc[1][r];
+            mine = pair[r];
           }
         }
+        const int64_t at = (int64_t)(begin + r0 + lane) * N + feature;
         if (GATED) {
           const float g = fminf(first, p.limit);
           const float u = fminf(fmaxf(second, -p.limit), p.limit);
-          ((__nv_bfloat16*)p.out)[(int64_t)(begin + r0 + lane) * N + feature] =
-              __float2bfloat16_rn(g / (1.f + expf(-p.slope * g)) * (u + p.up_offset));
+          ((__nv_bfloat16*)p.out)[at] = __float2bfloat16_rn(g / (1.f + expf(-p.slope * g)) * (u + p.up_offset));
         } else if (FIRST) {
-          ((__nv_bfloat16*)p.out)[(int64_t)(begin + r0 + lane) * N + feature] =
-              __float2bfloat16_rn(activation_value(first, p.activation));
+          ((__nv_bfloat16*)p.out)[at] = __float2bfloat16_rn(activation_value(first, p.activation));
+          if (pairs) ((__nv_bfloat16*)p.out)[at + 1] = __float2bfloat16_rn(activation_value(second, p.activation));
         } else {
-          int mine = pair[0];
-#pragma unroll
-          for (int r = 1; r < kGemvRows; ++r)
-            if (r == lane) mine = pair[r];
-          ((float*)p.out)[(int64_t)mine * N + feature] = p.weights[mine] * first;
+          float* dst = (float*)p.out + (int64_t)mine * N + feature;
+          const float weight = p.weights[mine];
+          dst[0] = weight * first;
+          if (pairs) dst[1] = weight * second;
         }
       }
     }

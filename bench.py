@@ -1,6 +1,6 @@
 """Benchmark of the engine on one B200: decode tokens per second at the Qwen3-8B shape.
 
-    python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--impl reference] [--shape 8b|14b|32b|sukalorn|zifuzen|renadra|zavizen|ligirax]
+    python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--impl reference] [--shape 8b|14b|32b|sukalorn|zifuzen|renadra|zavizen|ligirax|gosizen]
 
 Prints ONE JSON line.  A "step" is one decode step of the whole batch through the engine's own step
 function (every kernel of the model and the token choice); ``value`` is batch / step time, timed with CUDA
@@ -597,6 +597,48 @@ def ligirax_config(z: dict, layers: int, feed_forward: bool = True) -> dict:
         out[2]["mixer"]["kv_from"] = 1
     return {"architecture": "Ligirax", "vocab": SUKALORN_VOCAB, "width": z["width"], "norm": {"eps": 1e-6},
             "residual_mult": 0.5, "logit_scale": 2.0, "layers": out}
+
+
+# Gosizen at sizes that resemble a real model's layers: four layers (parallel, latent attention, parallel, latent
+# attention), all with dense feed-forwards without a gate (half again as wide as the gated ones of the same size, so that
+# the matrices are equal) and a token input of 256.  Each kind of layer also four times by itself beside its closest
+# design: parallel layers beside Renadra's (attention beside a linear memory, one output product), latent layers beside
+# Sukalorn's (latent attention behind a query latent, a dense feed-forward without a gate; over all keys), and parallel
+# layers with routed experts, which no other design has, by their kernels.
+GOSIZEN_SIZES = {
+    "2k": dict(width=2048, heads=16, kv_heads=4, dim=128, ff=8192, memory_heads=16, rot_dim=64, q_rank=768, kv_rank=512,
+               window=1024, block=1024, keep=64, rank=128, side=256, experts=32, top=6, expert_ff=1152),
+    "4k": dict(width=4096, heads=32, kv_heads=8, dim=128, ff=12288, memory_heads=32, rot_dim=64, q_rank=1536, kv_rank=512,
+               window=1024, block=1024, keep=64, rank=128, side=256, experts=64, top=6, expert_ff=1536),
+}
+
+
+def gosizen_config(z: dict, layers: int, kinds: tuple = ("parallel", "latent_attention")) -> dict:
+    d, h = z["dim"], z["memory_heads"]
+    left = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "conv": 4, "scale": d ** -0.5,
+            "mask": {"size": z["block"]},
+            "rot": {"base": 500000.0, "dims": d, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    right = {"heads": h, "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "conv": 4, "decay_rank": z["rank"],
+             "gate_rank": z["rank"]}
+    latent = {"heads": z["heads"], "dim": d, "rot_dim": z["rot_dim"], "vdim": d, "q_rank": z["q_rank"],
+              "kv_rank": z["kv_rank"], "scale": (d + z["rot_dim"]) ** -0.5, "mask": {"size": z["window"]},
+              "rot": {"base": 10000.0, "dims": z["rot_dim"]}}
+    mixers = {"parallel": {"left": left, "right": right, "left_scale": 0.8, "right_scale": 0.6}, "latent_attention": latent}
+    return {"architecture": "Gosizen", "vocab": SUKALORN_VOCAB, "width": z["width"], "norm": {"eps": 1e-6},
+            "logit_softcap": 30.0, "token_side": {"dim": z["side"]},
+            "layers": [{"type": kinds[i % len(kinds)], "mixer": json.loads(json.dumps(mixers[kinds[i % len(kinds)]])),
+                        "mlp": {"kind": "dense", "ff": z["ff"] * 3 // 2}} for i in range(layers)]}
+
+
+def gosizen_like_parallel(z: dict, layers: int) -> dict:
+    out = renadra_config(z, 4)
+    layer = out["layers"][2]
+    return dict(out, layers=[json.loads(json.dumps(layer)) for _ in range(layers)])
+
+
+def gosizen_like_latent(z: dict, layers: int) -> dict:
+    out = sukalorn_config(dict(z, ff=z["ff"] * 3 // 2), 2)
+    return dict(out, layers=[json.loads(json.dumps(out["layers"][1])) for _ in range(layers)])
 
 
 def ligirax_like_experts(z: dict, layers: int) -> dict:
@@ -1237,7 +1279,173 @@ def sukalorn_shape(args, design: str = "sukalorn") -> int:
                         hidden, pieces, ones, 1e-6, torch.bfloat16), moved=W * (4.0 * rows_used + tokens * 10.0))
         return out
 
+    def gosizen_kernels_alone(z: dict) -> dict:
+        """The kernels that came with the Gosizen design by themselves at this size, each beside the like kernel of
+        another design: attention in blocks of positions with sinks beside the capped and gated one (Sukalorn) and the
+        plain one, attention over shared rows with window, gates and sinks beside the one without sinks (Ligirax), the
+        convolutions with turn and cache write beside the turn and write alone, the delta rule with a decay per channel
+        beside the one per head (Zifuzen), the experts without a gate beside gated ones of equal FLOPs, gates and
+        activations of columns beside the activation of a whole matrix, and what acts on the stream beside the residual
+        add + RMS norm."""
+        out = {}
+        heads, kvh, dim, R, rank, W = z["heads"], z["kv_heads"], z["dim"], z["rot_dim"], z["kv_rank"], z["width"]
+        H, E, top, F, page, taps = z["memory_heads"], z["experts"], z["top"], z["expert_ff"], args.page_size, 4
+        row, block, window = rank + R, z["block"], z["window"]
+        bf = dict(dtype=torch.bfloat16, device=device)
+        g = torch.Generator(device=device).manual_seed(5)
+        dev = lambda v: torch.tensor(v, dtype=torch.int32, device=device)
+        fp32_peak = peaks.get("fp32_tflops") or FP32_FMA_TFLOPS
+
+        def record(key, fn, *, flops=0.0, moved=0.0, fp32=0.0):
+            for _ in range(3):
+                fn()
+            ms = timed(fn, 5, flush_l2=True)
+            entry = {"ms": round(ms, 4)}
+            if flops:
+                entry["tflops"] = round(flops / (ms / 1000) / 1e12, 2)
+                entry["frac_of_bf16_peak"] = round(flops / (ms / 1000) / 1e12 / peaks["bf16_tflops"], 4)
+            if fp32:
+                entry["fp32_tflops"] = round(fp32 / (ms / 1000) / 1e12, 3)
+                entry["frac_of_fp32_fma_peak"] = round(fp32 / (ms / 1000) / 1e12 / fp32_peak, 4)
+            if moved:
+                entry["gbs"] = round(moved / (ms / 1000) / 1e9, 1)
+                entry["frac_of_hbm"] = round(moved / (ms / 1000) / 1e9 / peaks["hbm_gbs"], 4)
+            out[key] = entry
+
+        for name, seq_q, q_tile in (("prompt", [(PREFILL_TOKENS, PREFILL_TOKENS)], ops.ATTENTION_Q_TILE),
+                                    ("decode", [(PROMPT_LEN, 1)] * batch, 1)):
+            lay, pages, tokens = layout(seq_q, q_tile)
+            rand = lambda *shape: torch.randn(shape, generator=g, **bf)
+            k_pages, v_pages, rows = rand(pages, kvh, page, dim), rand(pages, kvh, page, dim), rand(pages, 1, page, row)
+            q, q_row = rand(tokens, heads * dim), rand(tokens, heads * row)
+            sink, gate = torch.randn((heads,), device=device, generator=g), torch.rand((tokens, heads), device=device, generator=g)
+            slopes = torch.exp2(-8.0 * torch.arange(1, heads + 1, device=device) / heads).float()
+            group = heads // kvh
+            # blocks of positions: the prompt's tokens see half a block on average, the single tokens the whole of one
+            for case, chunk, extra in (("block_attention_sinks", block, dict(sink=sink)), ("like_block_attention", block, {}),
+                                       ("like_sukalorn_attention", 0, dict(softcap=30.0, slopes=slopes, gate=gate))):
+                seen = lambda p: p % chunk + 1 if chunk else p + 1
+                pairs = sum(seen(c - n + i) for c, n in seq_q for i in range(n))
+                keys = sum(seen(c - 1) for c, _ in seq_q)
+                splits = 1 if q_tile > 1 else ops.choose_splits(lay["num_tiles"], kvh, group, min(PROMPT_LEN, chunk or PROMPT_LEN), True)
+                record(f"{name}_{case}", lambda: ops.scored_attention(
+                    q, k_pages, v_pages, num_splits=splits, num_heads=heads, num_kv_heads=kvh, v_dim=dim, scale=dim ** -0.5,
+                    chunk=chunk, **extra, **lay), flops=4.0 * heads * dim * pairs, moved=2.0 * 2 * kvh * dim * keys)
+            for case, extra in (("latent_window_attention_sinks", dict(sink=sink)), ("like_latent_window_attention", {})):
+                pairs = sum(min(c - n + i + 1, window) for c, n in seq_q for i in range(n))
+                splits = ops.choose_splits_shared_rows(lay["num_tiles"], 1, q_tile * heads, min(max(c for c, _ in seq_q), window))
+                record(f"{name}_{case}", lambda: ops.scored_attention(
+                    q_row, rows, rows, num_splits=splits, num_heads=heads, num_kv_heads=1, v_dim=rank, scale=0.07,
+                    window=window, gate=gate, **extra, **lay), flops=2.0 * heads * (row + rank) * pairs,
+                    moved=2.0 * row * sum(min(c, window) for c, _ in seq_q))
+            # before attention
+            lens = [n for _, n in seq_q]
+            cu, slots = dev([0] + [sum(lens[:i + 1]) for i in range(len(lens))]), dev(list(range(len(lens))))
+            positions, at = dev([c - n + i for c, n in seq_q for i in range(n)]), dev(list(range(tokens)))
+            freq = torch.rand((dim // 2,), device=device, generator=g)
+            channels = (heads + 2 * kvh) * dim
+            width_in = channels + heads * dim
+            x = rand(tokens, width_in)
+            conv, bias = torch.rand((channels, taps), device=device, generator=g) - 0.3, torch.zeros((channels,), device=device)
+            tails = torch.zeros((batch + 1, (taps - 1) * channels), device=device)
+            prep = dict(num_heads=heads, num_kv_heads=kvh, head_dim=dim, v_dim=dim, rotary_dims=dim, layout="half")
+            record(f"{name}_conv_rotary_prep", lambda: ops.conv_rotary_prep(
+                x, conv, positions, at, freq, k_pages, v_pages, tails, cu, slots, taps=taps, bias=bias, **prep),
+                moved=4.0 * tokens * channels)
+            record(f"{name}_like_rotary_prep", lambda: ops.rotary_prep(x, positions, at, freq, k_pages, v_pages, **prep),
+                   moved=4.0 * tokens * channels)
+            heads_out, joined = rand(tokens, heads * dim), torch.empty((tokens, 2 * heads * dim + z["ff"] * 3 // 2), **bf)
+            record(f"{name}_gate_columns", lambda: ops.gate_columns(heads_out, x, channels, factor=0.8, out=joined),
+                   moved=6.0 * tokens * heads * dim)
+            ffw = z["ff"] * 3 // 2
+            up = rand(tokens, ffw + 64)
+            record(f"{name}_activation_columns", lambda: ops.activation_columns(up, 64, ffw, "gelu_tanh", out=joined,
+                                                                                out_off=2 * heads * dim), moved=4.0 * tokens * ffw)
+            up2 = rand(tokens, ffw)
+            record(f"{name}_like_activation", lambda: ops.activation(up2, "relu2"), moved=4.0 * tokens * ffw)
+            # the delta rule
+            G, D, V = kvh, dim, dim
+            dch = 2 * G * D + H * V
+            mem, floats = ops.delta_state_floats(H, G, D, V, taps)
+            state = torch.zeros((batch + 1, floats), device=device)
+            xd, xz = rand(tokens, dch + H), rand(tokens, dch + H * V + 2 * H)
+            mid = torch.randn((tokens, H * D + H * V), device=device, generator=g)
+            dconv = torch.rand((dch, taps), device=device, generator=g) - 0.3
+            rate, step_bias = torch.full((H,), -2.0, device=device), torch.zeros((H * D,), device=device)
+            ones_v, kw = torch.ones((V,), device=device), dict(num_heads=H, num_kv_heads=G, head_dim=D, v_dim=V, taps=taps)
+            chan = lambda: ops.delta_prep(xd, dconv, rate, step_bias, state, cu, slots, unit_eps=1e-6, steps=mid,
+                                          beta_off=dch, channel_decay=True, **kw)
+            head = lambda: ops.delta_prep(xz, dconv, rate, step_bias[:H].contiguous(), state, cu, slots, unit_eps=1e-6, **kw)
+            record(f"{name}_delta_prep_channel", chan, moved=tokens * (2.0 * (dch + H) + 4.0 * (dch + H + 2 * H * D)))
+            record(f"{name}_like_delta_prep", head, moved=tokens * (2.0 * (dch + 2 * H) + 4.0 * (dch + 2 * H)))
+            (qkv, coef), (zqkv, zcoef) = chan(), head()
+            ops_per, moved = 7.0 * tokens * H * D * V, 2.0 * 4 * len(lens) * mem
+            record(f"{name}_delta_scan_channel", lambda: ops.delta_scan(
+                qkv, coef, xd, ones_v, state, cu, slots, norm_eps=1e-6, gates=mid, gate_off=H * D, gate="sigmoid",
+                channel_decay=True, out=joined, out_off=heads * dim, **kw), fp32=ops_per, moved=moved)
+            record(f"{name}_like_delta_scan", lambda: ops.delta_scan(
+                zqkv, zcoef, xz, ones_v, state, cu, slots, norm_eps=1e-6, **kw), fp32=ops_per, moved=moved)
+            low, w_mid = rand(tokens, 2 * z["rank"] + 64), rand(H * D + H * V, 2 * z["rank"])
+            record(f"{name}_low_rank_product", lambda: ops.linear(low[:, :2 * z["rank"]], w_mid, out_dtype=torch.float32),
+                   flops=2.0 * tokens * w_mid.numel(), moved=2.0 * w_mid.numel() + tokens * 4.0 * (H * D + H * V))
+            # routed experts
+            logits, rbias = torch.randn((tokens, E), device=device, generator=g), torch.zeros((E,), device=device)
+            chosen, weights = ops.moe_route(logits, None, top=top, groups=1, keep_groups=1, group_top=1, scale=1.0,
+                                            weight_eps=0.0, score="softmax", bias=rbias)
+            order, offsets = ops.moe_sort(chosen, E)
+            used, n_rows = int((offsets[1:] > offsets[:-1]).sum()), tokens * top
+            h = rand(tokens, W)
+            w_up = (torch.randn((E, F, W), device=device, generator=g) * 0.02).to(torch.bfloat16)
+            w_gu = (torch.randn((E, 2 * (F // 2), W), device=device, generator=g) * 0.02).to(torch.bfloat16)
+            w_d = (torch.randn((E, W, F), device=device, generator=g) * 0.02).to(torch.bfloat16)
+            record(f"{name}_moe_up", lambda: ops.moe_up(h, w_up, order, offsets, top=top, activation="gelu"),
+                   flops=2.0 * n_rows * F * W, moved=2.0 * used * F * W)
+            record(f"{name}_like_moe_gate_up", lambda: ops.moe_gate_up(h, w_gu, order, offsets, top=top, limit=7.0, slope=1.702),
+                   flops=2.0 * n_rows * F * W, moved=2.0 * used * F * W)
+            act = ops.moe_up(h, w_up, order, offsets, top=top, activation="gelu")
+            parts = ops.moe_down(act, w_d, order, offsets, weights)
+            # the stream
+            hidden, ones = torch.randn((tokens, W), device=device, generator=g), torch.ones((W,), device=device)
+            start, y = torch.randn((tokens, W), device=device, generator=g), torch.randn((tokens, W), device=device, generator=g)
+            pieces = ops.ExpertParts(parts, None, top)
+            record(f"{name}_stream_sum", lambda: ops.stream_sum(hidden, [h], copy_dtype=torch.bfloat16), moved=tokens * W * 12.0)
+            record(f"{name}_stream_sum_experts", lambda: ops.stream_sum(hidden, [h, pieces], copy_dtype=torch.bfloat16),
+                   moved=tokens * W * (12.0 + 4.0 * top))
+            record(f"{name}_like_add_rmsnorm", lambda: ops.add_rmsnorm(hidden, h, ones, 1e-6, torch.bfloat16), moved=tokens * W * 12.0)
+            record(f"{name}_branch_rmsnorm", lambda: ops.branch_rmsnorm(hidden, ops.NormedBranch(y, ones, 1e-6), ones, 1e-6,
+                                                                        torch.bfloat16), moved=tokens * W * 14.0)
+            record(f"{name}_stream_concat", lambda: ops.stream_concat(hidden, start, torch.bfloat16), moved=tokens * W * 12.0)
+            record(f"{name}_stream_row_add", lambda: ops.stream_row_add(hidden, ones), moved=tokens * W * 8.0)
+            ids, table, zz = dev([i * 7 % 32000 for i in range(tokens)]), rand(32000, 4 * z["side"]), rand(tokens, z["side"])
+            record(f"{name}_token_gate", lambda: ops.token_gate(zz, ids, table, z["side"]), moved=tokens * 6.0 * z["side"])
+        return out
+
     sizes = {}
+    if design == "gosizen":
+        with ClockSampler() as clocks:
+            for name, z in GOSIZEN_SIZES.items():
+                sizes[name] = {"gosizen": measure(gosizen_config(z, layers)),
+                               "gosizen_parallel": measure(gosizen_config(z, layers, ("parallel",))),
+                               "renadra_parallel": measure(gosizen_like_parallel(z, layers)),
+                               "gosizen_latent": measure(gosizen_config(z, layers, ("latent_attention",))),
+                               "sukalorn_latent": measure(gosizen_like_latent(z, layers)),
+                               "kernels": gosizen_kernels_alone(z)}
+        head = sizes["4k"]["gosizen"]
+        line = {"metric": "decode tok/s at batch 8 of four Gosizen layers (width 4,096, B200); prefill, a smaller size, each "
+                          "kind of layer by itself beside Renadra's parallel and Sukalorn's latent layers of equal size, and "
+                          "Gosizen's kernels alone, each beside the like kernel of another design, alongside",
+                "value": head["decode_tok_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
+                "warmup": args.warmup, "ms_per_step": head["decode_ms"], "higher_is_better": True, "dtype": "bf16",
+                "data": "synthetic (seeded uniform token ids, seeded random weights)",
+                "config": {"model": "Gosizen", "layers": layers, "sizes": GOSIZEN_SIZES, "vocab": SUKALORN_VOCAB,
+                           "global_batch": batch, "prompt_len": PROMPT_LEN, "prefill_tokens": PREFILL_TOKENS,
+                           "page_size": args.page_size, "l2": "whole steps: inputs larger than L2; kernels alone: L2 "
+                           "flushed (a 256 MB write) before every timed launch", "peaks": peaks["source"],
+                           "fp32_fma_tflops": FP32_FMA_TFLOPS},
+                "gpu_launches": head["launches_per_decode_step"] * args.steps, "sizes": sizes,
+                "clocks": clocks.summary()}
+        print(json.dumps(line))
+        return 0
     if design == "ligirax":
         with ClockSampler() as clocks:
             for name, z in LIGIRAX_SIZES.items():
@@ -1351,7 +1559,7 @@ def main() -> int:
     parser.add_argument("--warmup", type=int, default=8)
     parser.add_argument("--impl", choices=("ours", "reference"), default="ours")
     parser.add_argument("--page-size", type=int, default=PAGE_SIZE, help="tokens per cache page (a power of two, 16 or more)")
-    parser.add_argument("--shape", choices=sorted(SHAPES) + ["ligirax", "renadra", "sukalorn", "zavizen", "zifuzen"], default="8b",
+    parser.add_argument("--shape", choices=sorted(SHAPES) + ["gosizen", "ligirax", "renadra", "sukalorn", "zavizen", "zifuzen"], default="8b",
                         help="8b: the headline benchmark; 14b: a mixed scheduler load of 64 requests; 32b: long-context "
                              "decode at batch 16; sukalorn: prefill and decode of the Sukalorn design at two layer "
                              "sizes beside Qwen3 layers of equal size; zifuzen: the same for the Zifuzen design; renadra: the Renadra design beside "
@@ -1364,7 +1572,7 @@ def main() -> int:
     parser.add_argument("--no-points", action="store_true", help="skip the batch-1 and batch-64 decode points")
     args = parser.parse_args()
 
-    if args.shape in ("ligirax", "renadra", "sukalorn", "zavizen", "zifuzen"):
+    if args.shape in ("gosizen", "ligirax", "renadra", "sukalorn", "zavizen", "zifuzen"):
         if args.impl == "reference":
             print(json.dumps({"impl": "reference", "unavailable": "the reference arm runs the 8b shape only"}))
             return 0

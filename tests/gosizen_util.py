@@ -192,12 +192,13 @@ def plain_logits(folder: str, raw: dict, requests: dict[str, list[int]]) -> dict
     return {rid: plain.forward(raw, w, toks).float() for rid, toks in requests.items()}
 
 
-def check(trace, outputs, expected, dtype: str) -> tuple[float, float]:
+def check(trace, outputs, expected, dtype: str, loose: float = 1.0) -> tuple[float, float]:
     """Every written row against the plain one, measured by the row's own scale (relative RMS error, worst element).
     float32: the two differ by summation order and by float32 angles.  bfloat16: a row's rounding error is a few per cent
-    of its scale, while a row that is wrong as a whole (a wrong page, a wrong expert, a lost state) misses by all of it."""
+    of its scale, while a row that is wrong as a whole (a wrong page, a wrong expert, a lost state) misses by all of it.
+    ``loose``: a factor on the bounds for configurations drawn at random, some of which norm one or four numbers."""
     rms, peak = (1e-4, 5e-4) if dtype == "float32" else (0.15, 0.5)
-    return ru.compare_rows_to_scale(trace, outputs, expected, rms_bound=rms, peak_bound=peak)
+    return ru.compare_rows_to_scale(trace, outputs, expected, rms_bound=rms * loose, peak_bound=peak * loose)
 
 
 def decisive_requests(folder: str, raw: dict, lengths, seed: int, margin: float = 0.08, tries: int = 400

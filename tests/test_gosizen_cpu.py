@@ -214,4 +214,4 @@ def test_random_configurations_replay(fake_ext, seed):
     expected = gu.plain_logits(folder, raw, requests)
     trace = ru.trace_mixed(requests, 64 * 4, seed=seed)
     outputs = ru.run_inprocess(folder, "float32", trace, 64 * 4, page_size=page)
-    gu.check(trace, outputs, expected, "float32")
+    gu.check(trace, outputs, expected, "float32", loose=5.0)
