@@ -81,8 +81,8 @@ __device__ __forceinline__ float activation_value(float z, int kind) {
     const float r = fmaxf(z, 0.f);
     return r * r;
   }
-  // (1 + tanh u) / 2 = 1 / (1 + e^(-2u)) and 1 + erf u = erfc(-u): no cancellation where z is far below zero
-  if (kind == 1) return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+  if (kind == 1) return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  // 1 + erf u = erfc(-u): no cancellation where z is far below zero
   if (kind == 3) return 0.5f * z * erfcf(-0.7071067811865476f * z);
   return z / (1.f + expf(-z));
 }

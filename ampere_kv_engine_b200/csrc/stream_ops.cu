@@ -183,6 +183,12 @@ __global__ void __launch_bounds__(256) stream_row_add_kernel(float* __restrict__
   *reinterpret_cast<float4*>(hidden + i) = h;
 }
 
+// The tanh form of GELU as z / (1 + e^(-2u)), (1 + tanh u) / 2 being 1 / (1 + e^(-2u)): what leaves here is divided by its
+// own root mean square later, so it keeps its relative precision far below zero too.
+__device__ __forceinline__ float gelu_tanh_tail(float z) {
+  return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
+
 template <typename T>
 __global__ void token_gate_kernel(TokenGateParams p) {
   pdl_launch_dependents();
@@ -198,7 +204,7 @@ __global__ void token_gate_kernel(TokenGateParams p) {
   const T* z = (const T*)p.z + token * p.dim;
   T* out = (T*)p.out + token * p.dim;
   for (int c = threadIdx.x; c < p.dim; c += blockDim.x)
-    out[c] = from_float<T>(activation_value(to_float<T>(z[c]), kActGeluTanh) * to_float<T>(e[c]));
+    out[c] = from_float<T>(gelu_tanh_tail(to_float<T>(z[c])) * to_float<T>(e[c]));
 }
 
 bool aligned16(const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; }

@@ -84,20 +84,23 @@ class GatedDelta(Mixer):
     def param_specs(self):
         h, n = self.hidden_size, self.names
         if self.low_rank is None:
-            low = {n["step"]: ParamSpec((self.num_heads, h)), n["gate"]: ParamSpec((self.v_width, h))}
+            step, gate = {n["step"]: ParamSpec((self.num_heads, h))}, {n["gate"]: ParamSpec((self.v_width, h))}
         else:
             a, g = int(self.low_rank["step"]), int(self.low_rank["gate"])
-            low = {n["step_in"]: ParamSpec((FREE_SIZE, h), free_size=a), n["step_out"]: ParamSpec((self.steps, FREE_SIZE), free_size=a),
-                   n["gate_in"]: ParamSpec((FREE_SIZE, h), free_size=g), n["gate_out"]: ParamSpec((self.v_width, FREE_SIZE), free_size=g)}
+            step = {n["step_in"]: ParamSpec((FREE_SIZE, h), free_size=a),
+                    n["step_out"]: ParamSpec((self.steps, FREE_SIZE), free_size=a)}
+            gate = {n["gate_in"]: ParamSpec((FREE_SIZE, h), free_size=g),
+                    n["gate_out"]: ParamSpec((self.v_width, FREE_SIZE), free_size=g)}
         return {
-            **low,
             n["q"]: ParamSpec((self.qk_width, h)), n["q_conv"]: ParamSpec((self.qk_width, self.taps), kind="vector", init="unit_interval"),
             n["k"]: ParamSpec((self.qk_width, h)), n["k_conv"]: ParamSpec((self.qk_width, self.taps), kind="vector", init="unit_interval"),
             n["v"]: ParamSpec((self.v_width, h)), n["v_conv"]: ParamSpec((self.v_width, self.taps), kind="vector", init="unit_interval"),
             n["beta"]: ParamSpec((self.num_heads, h)),
             n["rate_log"]: ParamSpec((self.num_heads,), kind="vector", init="around_zero"),
             n["norm"]: ParamSpec((self.v_dim,), kind="vector", init="norm"),
+            **step,
             n["step_bias"]: ParamSpec((self.steps,), kind="vector", init="around_zero"),
+            **gate,
             n["out"]: ParamSpec((h, self.v_width)),
         }
 
