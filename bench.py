@@ -16,6 +16,8 @@ Renadra's kernels alone beside the like kernels of the other designs.
 like kernels of the other designs.
 ``--shape ligirax`` sets four Ligirax layers beside Zifuzen attention layers with experts of equal size, Ligirax's mixers
 alone beside Sukalorn's latent mixers of equal size, and Ligirax's kernels alone beside the like kernels of those.
+``--shape gosizen`` sets four Gosizen layers, and each kind of layer by itself beside Renadra's parallel and Sukalorn's
+latent layers of equal size, and Gosizen's kernels alone beside the like kernels of other designs.
 ``--shape sukalorn`` prints a line of its own: prefill and decode of four Sukalorn layers at two sizes beside Qwen3
 layers of equal size, and the attention kernels alone.
 Between timed steps nothing is flushed: every step streams the whole model (16 GB at full depth) through
@@ -1564,7 +1566,8 @@ def main() -> int:
                              "decode at batch 16; sukalorn: prefill and decode of the Sukalorn design at two layer "
                              "sizes beside Qwen3 layers of equal size; zifuzen: the same for the Zifuzen design; renadra: the Renadra design beside "
                              "Zifuzen layers of equal size; zavizen: the Zavizen design beside Renadra layers of equal "
-                             "size; ligirax: the Ligirax design beside Zifuzen's experts and Sukalorn's latent mixer "
+                             "size; ligirax: the Ligirax design beside Zifuzen's experts and Sukalorn's latent mixer; "
+                             "gosizen: the Gosizen design beside Renadra's parallel and Sukalorn's latent layers "
                              "(each prints its own one line)")
     parser.add_argument("--layers", type=int, default=None,
                         help="run fewer layers of the same sizes (reported in config beside the full count)")
